@@ -429,10 +429,10 @@ qk_rotate_norm_store_kernel(T* __restrict__ rows, int row_elems, int H, int G, i
 // outputs, a warp an output: lanes stride over i, then a butterfly.
 constexpr int HL_TOK = 8, HL_WARPS = 8;
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(HL_WARPS * 32)
 head_linear_kernel(const T* __restrict__ x, int x_stride, int x_head, int x_off, const T* __restrict__ w,
-                   T* __restrict__ out, int o_stride, int o_head, int o_off, int n_tok, int I, int O) {
+                   TO* __restrict__ out, int o_stride, int o_head, int o_off, int n_tok, int I, int O) {
     extern __shared__ float hl_smem[];
     const int t0 = blockIdx.x * HL_TOK, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int n_here = min(HL_TOK, n_tok - t0);
@@ -457,7 +457,7 @@ head_linear_kernel(const T* __restrict__ x, int x_stride, int x_head, int x_off,
         for (int tt = 0; tt < HL_TOK; ++tt) {
             const float v = warp_sum(acc[tt]);
             if (lane == 0 && tt < n_here)
-                out[(size_t)(t0 + tt) * o_stride + (size_t)h * o_head + o_off + o] = from_float<T>(v);
+                out[(size_t)(t0 + tt) * o_stride + (size_t)h * o_head + o_off + o] = from_float<TO>(v);
         }
     }
 }
@@ -581,7 +581,7 @@ JANIS_EXPORT int janis_qk_rotate_norm_store(void* rows, int dtype, int row_elems
 }
 
 JANIS_EXPORT int janis_head_linear(const void* x, int dtype, int x_stride, int x_head, int x_off, const void* w, void* out,
-                                   int o_stride, int o_head, int o_off, int T, int H, int I, int O, cudaStream_t stream) {
+                                   int out_dtype, int o_stride, int o_head, int o_off, int T, int H, int I, int O, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || I <= 0 || O <= 0) return fail("head_linear: %d heads, %d -> %d", H, I, O);
     const size_t bytes = (size_t)HL_TOK * I * sizeof(float);
@@ -590,11 +590,14 @@ JANIS_EXPORT int janis_head_linear(const void* x, int dtype, int x_stride, int x
     if (gz > 65535) gz = 65535;
     if (H > 65535) return fail("head_linear: too many heads (%d)", H);
     const dim3 grid((T + HL_TOK - 1) / HL_TOK, H, gz), block(HL_WARPS * 32);
-    if (dtype == JANIS_F32)
-        return launch_kernel("head_linear", head_linear_kernel<float>, grid, block, bytes, stream, 1, (const float*)x, x_stride,
+    if (dtype == JANIS_F32 && out_dtype == JANIS_F32)
+        return launch_kernel("head_linear", head_linear_kernel<float, float>, grid, block, bytes, stream, 1, (const float*)x, x_stride,
                              x_head, x_off, (const float*)w, (float*)out, o_stride, o_head, o_off, T, I, O);
-    if (dtype == JANIS_BF16)
-        return launch_kernel("head_linear", head_linear_kernel<bf16>, grid, block, bytes, stream, 1, (const bf16*)x, x_stride,
+    if (dtype == JANIS_BF16 && out_dtype == JANIS_F32)
+        return launch_kernel("head_linear", head_linear_kernel<bf16, float>, grid, block, bytes, stream, 1, (const bf16*)x, x_stride,
+                             x_head, x_off, (const bf16*)w, (float*)out, o_stride, o_head, o_off, T, I, O);
+    if (dtype == JANIS_BF16 && out_dtype == JANIS_BF16)
+        return launch_kernel("head_linear", head_linear_kernel<bf16, bf16>, grid, block, bytes, stream, 1, (const bf16*)x, x_stride,
                              x_head, x_off, (const bf16*)w, (bf16*)out, o_stride, o_head, o_off, T, I, O);
-    return fail("head_linear: unknown dtype %d", dtype);
+    return fail("head_linear: unknown dtypes %d -> %d", dtype, out_dtype);
 }

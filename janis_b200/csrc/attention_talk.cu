@@ -28,19 +28,31 @@
 namespace janis {
 
 // ---------------------------------------------------------------------------
-// Rotary encoding of a step's queries and keys (first `rot` features, pairs i, i + rot/2), rotation of its
-// values over all dv features when inv_v is given, and the write of keys and values into the paged cache
+// Rotary encoding of a step's queries and keys (first `rot` features, pairs i, i + rot/2, sine and cosine times `amp`),
+// rotation of its values over all dv features when inv_v is given, and the write of keys and values into the paged cache
 // line.  A row of the step holds q (H heads of d), then k (G heads of d), then v (G heads of dv); a layer
-// that only reads a line has rows of q alone (with_kv == 0).  One CTA per token.
+// that only reads a line has rows of q alone (with_kv == 0).  With `bias` (floats, one per column of the row's q | k | v)
+// it is added first.  `mix` 1: the values are also left in v_first, as they are before they are stored; `mix` 2: the
+// values become (1 - share) v + share v_first.  One CTA per token; a pair's sine and cosine are formed once for all heads.
 // ---------------------------------------------------------------------------
+struct RotateExtras {
+    const float* bias;      // [H d + G d + G dv] (or the first H d of it), or null
+    float amp;              // on sine and cosine of the queries' and keys' turn
+    int mix;                // 0 none; 1 leave the values in v_first; 2 mix v_first in
+    float share;            // the weight of v_first
+};
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 qkv_rotate_store_kernel(T* __restrict__ rows, int row_elems, const int* __restrict__ tok_pos,
                         const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
                         const float* __restrict__ inv_qk, int rot, const float* __restrict__ inv_v, int H, int G, int d,
                         int dv, int with_kv, T* __restrict__ kpool, T* __restrict__ vpool,
-                        const int* __restrict__ page_table, int table_stride) {
-    const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+                        const int* __restrict__ page_table, int table_stride, RotateExtras ex, T* __restrict__ v_first) {
+    extern __shared__ float2 turn_s[];                // (sine, cosine) of the queries' and keys' pairs, then of the values'
+    const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5, nwarp = nt >> 5;
+    const int hq = rot >> 1, hv = inv_v != nullptr ? dv >> 1 : 0, n_heads = with_kv ? H + G : H;
+    float2* turn_v = turn_s + hq;
     grid_dependents_launch();
     const int pos = tok_pos[t];
     T* kdst = nullptr;
@@ -53,43 +65,54 @@ qkv_rotate_store_kernel(T* __restrict__ rows, int row_elems, const int* __restri
             vdst = vpool + ((size_t)page * G * JANIS_PAGE + pos % JANIS_PAGE) * dv;
         }
     }
+    for (int i = tid; i < hq + hv; i += nt) {
+        float s, c;
+        if (i < hq) {
+            sincosf((float)pos * inv_qk[i], &s, &c);
+            turn_s[i] = make_float2(s * ex.amp, c * ex.amp);
+        } else {
+            sincosf((float)pos * inv_v[i - hq], &s, &c);
+            turn_s[i] = make_float2(s, c);
+        }
+    }
+    __syncthreads();
     grid_dependency_wait();
     T* row = rows + (size_t)t * row_elems;
-    const int hq = rot >> 1, n_rot_heads = with_kv ? H + G : H;
-    for (int u = tid; u < n_rot_heads * hq; u += nt) {
-        const int head = u / hq, i = u % hq;
-        float s, c;
-        sincosf((float)pos * inv_qk[i], &s, &c);
+    for (int head = warp; head < n_heads; head += nwarp) {       // a warp a head
         T* p = row + (size_t)head * d;
-        float lo, hi;
-        rotate_pair(to_float(p[i]), to_float(p[i + hq]), s, c, lo, hi);
-        const T tl = from_float<T>(lo), th = from_float<T>(hi);
-        p[i] = tl;
-        p[i + hq] = th;
-        if (head >= H && kdst) {
-            T* kd = kdst + (size_t)(head - H) * JANIS_PAGE * d;
-            kd[i] = tl;
-            kd[i + hq] = th;
+        const float* b = ex.bias != nullptr ? ex.bias + (size_t)head * d : nullptr;
+        T* kd = head >= H && kdst != nullptr ? kdst + (size_t)(head - H) * JANIS_PAGE * d : nullptr;
+        for (int i = lane; i < hq; i += 32) {
+            float x0 = to_float(p[i]), x1 = to_float(p[i + hq]);
+            if (b != nullptr) { x0 += b[i]; x1 += b[i + hq]; }
+            float lo, hi;
+            rotate_pair(x0, x1, turn_s[i].x, turn_s[i].y, lo, hi);
+            const T tl = from_float<T>(lo), th = from_float<T>(hi);
+            p[i] = tl;
+            p[i + hq] = th;
+            if (kd != nullptr) {
+                kd[i] = tl;
+                kd[i + hq] = th;
+            }
         }
+        if (b != nullptr || kd != nullptr)
+            for (int i = rot + lane; i < d; i += 32) {           // what does not turn
+                T x = p[i];
+                if (b != nullptr) {
+                    x = from_float<T>(to_float(x) + b[i]);
+                    p[i] = x;
+                }
+                if (kd != nullptr) kd[i] = x;
+            }
     }
     if (!with_kv) return;
-    if (kdst && rot < d) {
-        const int rest = d - rot;
-        for (int u = tid; u < G * rest; u += nt) {
-            const int g = u / rest, c = rot + u % rest;
-            kdst[(size_t)g * JANIS_PAGE * d + c] = row[(size_t)(H + g) * d + c];
-        }
-    }
     T* vrow = row + (size_t)(H + G) * d;
     if (inv_v != nullptr) {
-        const int hv = dv >> 1;
         for (int u = tid; u < G * hv; u += nt) {
             const int g = u / hv, m = u % hv;
-            float s, c;
-            sincosf((float)pos * inv_v[m], &s, &c);
             T* p = vrow + (size_t)g * dv;
             float lo, hi;
-            rotate_pair(to_float(p[m]), to_float(p[m + hv]), s, c, lo, hi);
+            rotate_pair(to_float(p[m]), to_float(p[m + hv]), turn_v[m].x, turn_v[m].y, lo, hi);
             const T tl = from_float<T>(lo), th = from_float<T>(hi);
             p[m] = tl;
             p[m + hv] = th;
@@ -99,9 +122,24 @@ qkv_rotate_store_kernel(T* __restrict__ rows, int row_elems, const int* __restri
                 vd[m + hv] = th;
             }
         }
-    } else if (vdst) {
-        for (int u = tid; u < G * dv; u += nt) vdst[(size_t)(u / dv) * JANIS_PAGE * dv + u % dv] = vrow[u];
+        return;
     }
+    const float* vb = ex.bias != nullptr ? ex.bias + (size_t)(H + G) * d : nullptr;
+    const bool touched = vb != nullptr || ex.mix != 0;
+    for (int g = warp; g < G; g += nwarp)
+        for (int c = lane; c < dv; c += 32) {
+            const int u = g * dv + c;
+            T x = vrow[u];
+            if (touched) {
+                float v = to_float(x);
+                if (vb != nullptr) v += vb[u];
+                if (ex.mix == 2) v = fmaf(ex.share, to_float(v_first[(size_t)t * G * dv + u]), (1.f - ex.share) * v);
+                x = from_float<T>(v);
+                vrow[u] = x;
+                if (ex.mix == 1) v_first[(size_t)t * G * dv + u] = x;
+            }
+            if (vdst) vdst[(size_t)g * JANIS_PAGE * dv + c] = x;
+        }
 }
 
 // ---------------------------------------------------------------------------
@@ -796,21 +834,27 @@ using namespace janis;
 JANIS_EXPORT int janis_qkv_rotate_store(void* rows, int dtype, int row_elems, const int* tok_pos, const int* tok_seq,
                                         const int* seq_slot, const float* inv_qk, int rot, const float* inv_v, int T,
                                         int H, int G, int d, int dv, int with_kv, void* kpool, void* vpool,
-                                        const int* page_table, int table_stride, cudaStream_t stream) {
+                                        const int* page_table, int table_stride, const float* bias, float amp, int mix,
+                                        float share, void* v_first, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (rot < 0 || rot > d || (rot & 1)) return fail("qkv_rotate_store: rotary width %d does not fit key size %d", rot, d);
     if (inv_v != nullptr && (dv & 1)) return fail("qkv_rotate_store: rotated values need an even size, found %d", dv);
     if (row_elems < H * d + (with_kv ? G * (d + dv) : 0)) return fail("qkv_rotate_store: rows of %d elements are too short", row_elems);
     if (with_kv && (!kpool || !vpool || !page_table || !seq_slot)) return fail("qkv_rotate_store: no cache line to store into");
+    if (mix < 0 || mix > 2 || (mix && (!with_kv || v_first == nullptr))) return fail("qkv_rotate_store: mixed values need values and a buffer of the first layer's");
+    if (inv_v != nullptr && (mix || bias != nullptr)) return fail("qkv_rotate_store: turned values take no bias and no mixing");
+    const size_t bytes = ((size_t)(rot >> 1) + (inv_v != nullptr ? dv >> 1 : 0)) * sizeof(float2);
+    if (bytes > 48 * 1024) return fail("qkv_rotate_store: %zu bytes of angles", bytes);
+    const RotateExtras ex = {bias, amp, mix, share};
     const dim3 grid(T), block(128);
     if (dtype == JANIS_F32)
-        return launch_kernel("qkv_rotate_store", qkv_rotate_store_kernel<float>, grid, block, 0, stream, 1, (float*)rows,
+        return launch_kernel("qkv_rotate_store", qkv_rotate_store_kernel<float>, grid, block, bytes, stream, 1, (float*)rows,
                              row_elems, tok_pos, tok_seq, seq_slot, inv_qk, rot, inv_v, H, G, d, dv, with_kv, (float*)kpool,
-                             (float*)vpool, page_table, table_stride);
+                             (float*)vpool, page_table, table_stride, ex, (float*)v_first);
     if (dtype == JANIS_BF16)
-        return launch_kernel("qkv_rotate_store", qkv_rotate_store_kernel<bf16>, grid, block, 0, stream, 1, (bf16*)rows,
+        return launch_kernel("qkv_rotate_store", qkv_rotate_store_kernel<bf16>, grid, block, bytes, stream, 1, (bf16*)rows,
                              row_elems, tok_pos, tok_seq, seq_slot, inv_qk, rot, inv_v, H, G, d, dv, with_kv, (bf16*)kpool,
-                             (bf16*)vpool, page_table, table_stride);
+                             (bf16*)vpool, page_table, table_stride, ex, (bf16*)v_first);
     return fail("qkv_rotate_store: unknown dtype %d", dtype);
 }
 

@@ -169,7 +169,7 @@ sigmoid_gate_kernel(T* __restrict__ x, const T* __restrict__ rows, int row_elems
 // Mixture of experts: the router and the experts' activation.
 //
 // router, a warp per token over E logits z (float):  s = sigmoid(z), c = s + correction;  experts form n_groups equal
-// groups of neighbours, a group's score is the sum of its two largest c, the best `keep` groups stay (ties: the
+// groups of neighbours, a group's score is the sum of its two largest c (group_best: its largest), the best `keep` groups stay (ties: the
 // lower index); among their experts the `top` of largest c are chosen (ties: the lower index); the chosen get
 // w_e = s_e / (sum of the chosen s + 1e-20) * scale, every other expert 0.  With a shared gate, column E of z is
 // its logit and column E of the output its sigmoid.  With `softmax` the scores are the softmax of z over all entries instead.  With
@@ -189,7 +189,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& at) {
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ z, const float* __restrict__ correction, int T, int E, int n_groups, int keep,
-                 int top, float scale, int shared_gate, float* __restrict__ out, int n_identity, int softmax) {
+                 int top, float scale, int shared_gate, float* __restrict__ out, int n_identity, int softmax, int group_best) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * ROUTE_WARPS + warp;
     const int N = E + n_identity;                    // entries the router scores: the experts, then the identity entries
@@ -217,7 +217,7 @@ moe_route_kernel(const float* __restrict__ z, const float* __restrict__ correcti
     for (int e = lane; e < N; e += 32) {
         const float v = softmax ? s[e] / zsum : 1.0f / (1.0f + expf(-zr[e]));
         s[e] = v;
-        c[e] = v + correction[e];
+        c[e] = correction != nullptr ? v + correction[e] : v;
         mark[e] = 0.f;
     }
     if (shared_gate && lane == 0) o[E] = 1.0f / (1.0f + expf(-zr[N]));
@@ -230,7 +230,7 @@ moe_route_kernel(const float* __restrict__ z, const float* __restrict__ correcti
                 if (v > a) { b = a; a = v; }
                 else if (v > b) b = v;
             }
-            gs[g] = per > 1 ? a + b : a;
+            gs[g] = per > 1 && !group_best ? a + b : a;
         }
         __syncwarp();
         // the kept groups get +inf as a mark; the others' experts leave the running
@@ -378,6 +378,69 @@ moe_expert_act_vec_kernel(const T* __restrict__ gu, const float* __restrict__ wt
     }
 }
 
+// x[t, col] = w[t, e] relu(x[t, col])^2 in place over the columns of all experts side by side (expert e: `ff` columns; then
+// the shared expert's `shared_ff`, whose weight is column E of the weights or, without one (shared_col == 0), 1).
+// Experts of weight 0 give exact zeros.  VEC: 16 bytes of columns a thread, all of one expert.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+moe_relu2_kernel(T* __restrict__ x, const float* __restrict__ wts, int E, int ff, int shared_ff, int shared_col, int T_rows,
+                 int wcols) {
+    constexpr int V = VEC ? Vec16<T>::N : 1;
+    const int total = E * ff + shared_ff, per_row = total / V;
+    grid_dependents_launch();
+    grid_dependency_wait();
+    for (int t = blockIdx.y; t < T_rows; t += gridDim.y) {
+        const float* wrow = wts + (size_t)t * wcols;
+        T* row = x + (size_t)t * total;
+        for (int ch = blockIdx.x * blockDim.x + threadIdx.x; ch < per_row; ch += gridDim.x * blockDim.x) {
+            const int col = ch * V;
+            const float w = col < E * ff ? wrow[col / ff] : (shared_col ? wrow[E] : 1.f);
+            float a[V];
+            if constexpr (VEC) {
+                if (w != 0.f) Vec16<T>::load(row + col, a);
+#pragma unroll
+                for (int i = 0; i < V; ++i) a[i] = w != 0.f && a[i] > 0.f ? w * a[i] * a[i] : 0.f;
+                Vec16<T>::store(row + col, a);
+            } else {
+                const float v = to_float(row[col]);
+                row[col] = from_float<T>(w != 0.f && v > 0.f ? w * v * v : 0.f);
+            }
+        }
+    }
+}
+
+// dst[t, d_off + c] = scale * x[t, c] * sigmoid(rows[t, g_off + c / per]) (no gate where rows is null): an attention's
+// heads on their way into the input of an output product that other branches share.  VEC: 16 bytes a thread (per == 1).
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+gate_place_kernel(const T* __restrict__ x, const T* __restrict__ rows, int row_elems, int g_off, int per, T* __restrict__ dst,
+                  int dst_elems, int d_off, float scale, int width, size_t n) {
+    constexpr int V = VEC ? Vec16<T>::N : 1;
+    grid_dependents_launch();
+    grid_dependency_wait();
+    for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V; i < n; i += (size_t)gridDim.x * blockDim.x * V) {
+        const size_t t = i / width;
+        const int c = (int)(i % width);
+        if constexpr (VEC) {
+            float a[V], g[V];
+            Vec16<T>::load(x + i, a);
+            if (rows != nullptr) {
+                Vec16<T>::load(rows + t * row_elems + g_off + c, g);
+#pragma unroll
+                for (int e = 0; e < V; ++e) a[e] = scale * (a[e] / (1.0f + expf(-g[e])));
+            } else {
+#pragma unroll
+                for (int e = 0; e < V; ++e) a[e] *= scale;
+            }
+            Vec16<T>::store(dst + t * dst_elems + d_off + c, a);
+        } else {
+            float a = to_float(x[i]);
+            if (rows != nullptr) a /= 1.0f + expf(-to_float(rows[t * row_elems + g_off + c / per]));
+            dst[t * dst_elems + d_off + c] = from_float<T>(scale * a);
+        }
+    }
+}
+
 }  // namespace janis
 
 using namespace janis;
@@ -475,7 +538,8 @@ JANIS_EXPORT int janis_round_rows(const float* h, void* y, size_t n, cudaStream_
 }
 
 JANIS_EXPORT int janis_moe_route(const float* z, const float* correction, int T, int E, int n_groups, int keep, int top,
-                                 float scale, int shared_gate, float* out, int n_identity, int softmax, cudaStream_t stream) {
+                                 float scale, int shared_gate, float* out, int n_identity, int softmax, int group_best,
+                                 cudaStream_t stream) {
     if (T <= 0) return 0;
     const int N = E + n_identity;
     if (E < 0 || n_identity < 0 || N <= 0 || N > 1024) return fail("moe_route: %d experts and %d identity entries (up to 1024 are taken)", E, n_identity);
@@ -484,7 +548,7 @@ JANIS_EXPORT int janis_moe_route(const float* z, const float* correction, int T,
         return fail("moe_route: %d entries in %d groups, %d kept, %d chosen", N, n_groups, keep, top);
     const size_t bytes = (size_t)ROUTE_WARPS * 4 * N * sizeof(float);
     return launch_kernel("moe_route", moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32),
-                         bytes, stream, 1, z, correction, T, E, n_groups, keep, top, scale, shared_gate, out, n_identity, softmax);
+                         bytes, stream, 1, z, correction, T, E, n_groups, keep, top, scale, shared_gate, out, n_identity, softmax, group_best);
 }
 
 JANIS_EXPORT int janis_moe_identity_add(void* out, const void* y, int dtype, const float* wts, int wts_stride, int w_col, int T,
@@ -525,4 +589,54 @@ JANIS_EXPORT int janis_moe_expert_act(const void* gu, int dtype, const float* wt
         return launch_kernel("moe_expert_act", moe_expert_act_kernel<bf16>, dim3(flat_grid(n)), dim3(256), 0, stream, 1,
                              (const bf16*)gu, wts, E, ff, limit, shared_ff, shared_limit, alpha, (bf16*)out, n, wts_stride, up_add);
     return fail("moe_expert_act: unknown dtype %d", dtype);
+}
+
+JANIS_EXPORT int janis_moe_relu2(void* x, int dtype, const float* wts, int wts_stride, int E, int ff, int shared_ff,
+                                 int shared_col, int T, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    const int total = E * ff + shared_ff;
+    if (total <= 0) return fail("moe_relu2: no columns (%d experts of %d, shared %d)", E, ff, shared_ff);
+    if (E + (shared_col ? 1 : 0) > wts_stride) return fail("moe_relu2: %d weights a row for %d experts", wts_stride, E);
+    const int v = dtype == JANIS_F32 ? 4 : 8;
+    const bool vec = ff % v == 0 && shared_ff % v == 0 && ((uintptr_t)x & 15) == 0;
+    const int per_row = vec ? total / v : total;
+    const dim3 grid((per_row + 255) / 256, T < 65535 ? T : 65535), block(256);
+#define JANIS_RELU2(TT, VEC)                                                                                           \
+    return launch_kernel("moe_relu2", moe_relu2_kernel<TT, VEC>, grid, block, 0, stream, 1, (TT*)x, wts, E, ff, shared_ff, \
+                         shared_col, T, wts_stride);
+    if (dtype == JANIS_F32) {
+        if (vec) JANIS_RELU2(float, true)
+        JANIS_RELU2(float, false)
+    }
+    if (dtype == JANIS_BF16) {
+        if (vec) JANIS_RELU2(bf16, true)
+        JANIS_RELU2(bf16, false)
+    }
+#undef JANIS_RELU2
+    return fail("moe_relu2: unknown dtype %d", dtype);
+}
+
+JANIS_EXPORT int janis_gate_place(const void* x, const void* rows, int dtype, int row_elems, int g_off, int per, void* dst,
+                                  int dst_elems, int d_off, float scale, int T, int width, cudaStream_t stream) {
+    if (T <= 0 || width <= 0) return 0;
+    if (per <= 0 || width % per) return fail("gate_place: runs of %d elements do not divide %d", per, width);
+    if (rows != nullptr && (g_off < 0 || g_off + width / per > row_elems)) return fail("gate_place: %d gates at %d do not fit rows of %d", width / per, g_off, row_elems);
+    if (d_off < 0 || d_off + width > dst_elems) return fail("gate_place: %d columns at %d do not fit rows of %d", width, d_off, dst_elems);
+    const size_t n = (size_t)T * width;
+    const int v = dtype == JANIS_F32 ? 4 : 8;
+    const bool vec = width % v == 0 && d_off % v == 0 && dst_elems % v == 0 && (((uintptr_t)x | (uintptr_t)dst) & 15) == 0 &&
+                     (rows == nullptr || (per == 1 && g_off % v == 0 && row_elems % v == 0 && ((uintptr_t)rows & 15) == 0));
+#define JANIS_PLACE(TT, VEC)                                                                                           \
+    return launch_kernel("gate_place", gate_place_kernel<TT, VEC>, dim3(flat_grid(VEC ? n / v : n)), dim3(256), 0, stream, 1, \
+                         (const TT*)x, (const TT*)rows, row_elems, g_off, per, (TT*)dst, dst_elems, d_off, scale, width, n);
+    if (dtype == JANIS_F32) {
+        if (vec) JANIS_PLACE(float, true)
+        JANIS_PLACE(float, false)
+    }
+    if (dtype == JANIS_BF16) {
+        if (vec) JANIS_PLACE(bf16, true)
+        JANIS_PLACE(bf16, false)
+    }
+#undef JANIS_PLACE
+    return fail("gate_place: unknown dtype %d", dtype);
 }

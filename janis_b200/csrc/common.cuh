@@ -207,6 +207,12 @@ __device__ __forceinline__ float gelu_tanh(float v) {
     return 0.5f * v * (1.0f + tanhf(inner));
 }
 
+// The clamped gate: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + up_add)
+__device__ __forceinline__ float clamped_gate(float gate, float up, float limit, float alpha, float up_add) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-alpha * g)) * (u + up_add);
+}
+
 // Activations of a dense feed-forward, by the codes of bias_act: 0 nothing; 1 xIELU with a_pos = softplus(p) and
 // a_neg = 1/2 + softplus(q) formed on the host (z > 0: a_pos z^2 + z/2; z <= 0: a_neg (e^z - 1 - z) + z/2);
 // 2 the tanh form of gelu; 3 silu; 4 the square of relu.

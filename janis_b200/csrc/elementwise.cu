@@ -189,11 +189,12 @@ add_rmsnorm_vec_kernel(float* __restrict__ h, const TR* __restrict__ res, int n_
 // ---------------------------------------------------------------------------
 // gated activation over a fused [rows, 2*I] product whose columns alternate in
 // groups of `group`: group g of gate columns, then group g of up columns.
-// act: 0 = gelu (tanh form), 1 = silu
+// act: 0 = gelu (tanh form), 1 = silu, 2 = the clamped gate: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g sigmoid(alpha g) (u + up_add)
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, int rows, int I, int group,
-                                 int act) {
+                                 int act, float limit, float alpha, float up_add) {
     grid_dependents_launch();
     grid_dependency_wait();
     const size_t n = (size_t)rows * I;
@@ -202,6 +203,10 @@ __global__ void gated_act_kernel(const T* __restrict__ gu, T* __restrict__ out, 
         const int r = (int)(idx / I), j = (int)(idx % I);
         const size_t base = (size_t)r * 2 * I + (size_t)(j / group) * 2 * group + (j % group);
         const float g = to_float(gu[base]), u = to_float(gu[base + group]);
+        if (act == 2) {
+            out[idx] = from_float<T>(clamped_gate(g, u, limit, alpha, up_add));
+            continue;
+        }
         const float a = act == 0 ? gelu_tanh(g) : g / (1.0f + expf(-g));
         out[idx] = from_float<T>(a * u);
     }
@@ -232,7 +237,8 @@ __device__ __forceinline__ float silu_fast(float v) {
 
 template <int ACT>
 __global__ void __launch_bounds__(256)
-gated_act8_bf16_kernel(const bf16* __restrict__ gu, bf16* __restrict__ out, size_t n_groups) {
+gated_act8_bf16_kernel(const bf16* __restrict__ gu, bf16* __restrict__ out, size_t n_groups, float limit, float alpha,
+                       float up_add) {
     grid_dependents_launch();
     grid_dependency_wait();
     for (size_t q = (size_t)blockIdx.x * blockDim.x + threadIdx.x; q < n_groups; q += (size_t)gridDim.x * blockDim.x) {
@@ -240,7 +246,14 @@ gated_act8_bf16_kernel(const bf16* __restrict__ gu, bf16* __restrict__ out, size
         Vec16<bf16>::load(gu + q * 16, g);
         Vec16<bf16>::load(gu + q * 16 + 8, u);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = (ACT == 0 ? gelu_tanh_fast(g[e]) : silu_fast(g[e])) * u[e];
+        for (int e = 0; e < 8; ++e) {
+            if constexpr (ACT == 2) {
+                const float gg = fminf(g[e], limit), uu = fminf(fmaxf(u[e], -limit), limit);
+                o[e] = gg * rcp_fast(1.0f + ex2_fast(-alpha * gg * 1.4426950408889634f)) * (uu + up_add);
+            } else {
+                o[e] = (ACT == 0 ? gelu_tanh_fast(g[e]) : silu_fast(g[e])) * u[e];
+            }
+        }
         Vec16<bf16>::store(out + q * 8, o);
     }
 }
@@ -568,29 +581,33 @@ JANIS_EXPORT int janis_add_rmsnorm(float* h, const void* res, int res_dtype, int
     return fail("add_rmsnorm: unknown dtypes %d -> %d", res_dtype, y_dtype);
 }
 
-JANIS_EXPORT int janis_gated_act(const void* gu, void* out, int dtype, int rows, int I, int group, int act,
-                                 cudaStream_t stream) {
+JANIS_EXPORT int janis_gated_act(const void* gu, void* out, int dtype, int rows, int I, int group, int act, float limit,
+                                 float alpha, float up_add, cudaStream_t stream) {
     if (rows <= 0) return 0;
+    if (act < 0 || act > 2) return fail("gated_act: unknown activation %d", act);
     if (group <= 0 || I % group) return fail("gated_act: width %d is not a multiple of the group %d", I, group);
     const size_t n = (size_t)rows * I;
     const int nt = 256;
     const int nb = (int)((n + nt - 1) / nt < 148 * 16 ? (n + nt - 1) / nt : 148 * 16);
     if (dtype == JANIS_F32)
         return launch_kernel("gated_act", gated_act_kernel<float>, dim3(nb), dim3(nt), 0, stream, 1, (const float*)gu,
-                             (float*)out, rows, I, group, act);
+                             (float*)out, rows, I, group, act, limit, alpha, up_add);
     if (dtype == JANIS_BF16 && group == 8 && (((uintptr_t)gu | (uintptr_t)out) & 15) == 0) {
         const size_t n_groups = n / 8;        // rows * I / 8: group q of a row-major [rows, 2I] starts at 16 q
         const size_t want = (n_groups + nt - 1) / nt;
         const dim3 grid((int)(want < 148 * 32 ? want : 148 * 32));
         if (act == 0)
             return launch_kernel("gated_act", gated_act8_bf16_kernel<0>, grid, dim3(nt), 0, stream, 1, (const bf16*)gu,
-                                 (bf16*)out, n_groups);
+                                 (bf16*)out, n_groups, limit, alpha, up_add);
+        if (act == 2)
+            return launch_kernel("gated_act", gated_act8_bf16_kernel<2>, grid, dim3(nt), 0, stream, 1, (const bf16*)gu,
+                                 (bf16*)out, n_groups, limit, alpha, up_add);
         return launch_kernel("gated_act", gated_act8_bf16_kernel<1>, grid, dim3(nt), 0, stream, 1, (const bf16*)gu,
-                             (bf16*)out, n_groups);
+                             (bf16*)out, n_groups, limit, alpha, up_add);
     }
     if (dtype == JANIS_BF16)
         return launch_kernel("gated_act", gated_act_kernel<bf16>, dim3(nb), dim3(nt), 0, stream, 1, (const bf16*)gu,
-                             (bf16*)out, rows, I, group, act);
+                             (bf16*)out, rows, I, group, act, limit, alpha, up_add);
     return fail("gated_act: unknown dtype %d", dtype);
 }
 

@@ -48,7 +48,8 @@ namespace janis {
 
 constexpr int GEMV_WARPS = 8;        // warps of a CTA that split K (4 when N alone gives CTAs enough)
 
-enum { EPI_NONE = 0, EPI_GATED_GELU = 1, EPI_SOFTCAP = 2, EPI_GATED_SILU = 3 };
+enum { EPI_NONE = 0, EPI_GATED_GELU = 1, EPI_SOFTCAP = 2, EPI_GATED_SILU = 3, EPI_GATED_CLAMP = 4 };   // (4: cap is the limit, BiasAct's
+                                      // two numbers are alpha and what is added to the up value)
 
 // What the ROPE variant needs beside the product: the step's tables, the inverse frequencies and one cache line.
 struct RopeStore {
@@ -335,7 +336,7 @@ gemv_bf16_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, TO* __r
         return;
     }
 
-    if (epi == EPI_GATED_GELU || epi == EPI_GATED_SILU) {
+    if (epi == EPI_GATED_GELU || epi == EPI_GATED_SILU || epi == EPI_GATED_CLAMP) {
         // rows g of the tile are gate rows, rows g + 8 the matching up rows
         const int I = N / 2;
         for (int idx = threadIdx.x; idx < MT * 32 * 2; idx += blockDim.x) {
@@ -344,8 +345,10 @@ gemv_bf16_kernel(const bf16* __restrict__ x, const bf16* __restrict__ W, TO* __r
             const int m = i * 8 + (ln & 3) * 2 + p;
             const int j = tile * 8 + (ln >> 2);
             if (m < M && j < I) {
-                const float a = epi == EPI_GATED_GELU ? gelu_tanh(gate) : gate / (1.0f + expf(-gate));
-                out[(size_t)m * I + j] = from_float<TO>(a * up);
+                float v;
+                if (epi == EPI_GATED_CLAMP) v = clamped_gate(gate, up, cap, ba.a_pos, ba.a_neg);
+                else v = (epi == EPI_GATED_GELU ? gelu_tanh(gate) : gate / (1.0f + expf(-gate))) * up;
+                out[(size_t)m * I + j] = from_float<TO>(v);
             }
         }
         return;
@@ -424,14 +427,14 @@ static int choose_cluster(int tiles, int nblk) {
 // x [M, K] bf16, W [N, K] bf16, out [M, N] (or [M, N/2] with a gated epilogue).
 // cluster: CTAs that share a tile's K (1, 2 or 4); 0 lets the kernel choose from N and K.
 JANIS_EXPORT int janis_gemv_bf16(const void* x, const void* W, void* out, int out_dtype, int M, int N, int K,
-                                 int epi, float cap, int cluster, cudaStream_t stream) {
+                                 int epi, float cap, int cluster, float alpha, float up_add, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > 64) return fail("gemv_bf16: at most 64 rows, found %d", M);
     if (K <= 0 || K % 8) return fail("gemv_bf16: K must be a positive multiple of 8, found %d", K);
     if (out_dtype != JANIS_BF16 && out_dtype != JANIS_F32) return fail("gemv_bf16: unknown output dtype %d", out_dtype);
-    if ((epi == EPI_GATED_GELU || epi == EPI_GATED_SILU) && N % 16)
+    if ((epi == EPI_GATED_GELU || epi == EPI_GATED_SILU || epi == EPI_GATED_CLAMP) && N % 16)
         return fail("gemv_bf16: a gated epilogue needs N to be a multiple of 16, found %d", N);
-    if (epi < 0 || epi > 3) return fail("gemv_bf16: unknown epilogue %d", epi);
+    if (epi < 0 || epi > 4) return fail("gemv_bf16: unknown epilogue %d", epi);
     if (cluster != 0 && cluster != 1 && cluster != 2 && cluster != 4)
         return fail("gemv_bf16: cluster must be 0, 1, 2 or 4, found %d", cluster);
     if (((uintptr_t)x | (uintptr_t)W) & 15) return fail("gemv_bf16: operands must be 16-byte aligned");
@@ -439,10 +442,11 @@ JANIS_EXPORT int janis_gemv_bf16(const void* x, const void* W, void* out, int ou
     const bf16* wp = (const bf16*)W;
     const int tiles = (N + 15) / 16, nblk = (K + 31) / 32;
     if (cluster == 0) cluster = choose_cluster(tiles, nblk);
-    if (M <= 8) return launch_gemv<1, JANIS_GEMV_U1>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream);
-    if (M <= 16) return launch_gemv<2, 4>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream);
-    if (M <= 32) return launch_gemv<4, 2>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream);
-    return launch_gemv<8, 1>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream);
+    const BiasAct ba = {nullptr, 0, alpha, up_add};
+    if (M <= 8) return launch_gemv<1, JANIS_GEMV_U1>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream, ba);
+    if (M <= 16) return launch_gemv<2, 4>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream, ba);
+    if (M <= 32) return launch_gemv<4, 2>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream, ba);
+    return launch_gemv<8, 1>(xp, wp, out, out_dtype, M, N, K, epi, cap, cluster, stream, ba);
 }
 
 // The same product with a bias (may be null) and an activation of a dense feed-forward (the codes of bias_act) in its

@@ -1,7 +1,8 @@
 // State-space mixers: a causal convolution per channel with silu, the selective scan, and the gated norm that
 // follows the scan of the state-space-duality form.
 //
-//   conv:  x'[t, c] = silu(b[c] + sum_j w[c, K-1-j] x[t-j, c])      inputs before the sequence's start are zero;
+//   conv:  x'[t, c] = silu(b[c] + sum_j w[c, K-1-j] x[t-j, c])      inputs before the sequence's start are zero (an
+//          input bias is part of x, so it is missing there too);
 //          the last K-1 inputs of a sequence are kept per slot, so that a later step goes on from them
 //   scan:  S[c, n] <- exp(delta A) S[c, n] + delta u[c] B[n];   o[c] = sum_n S[c, n] C[n] + D u[c]
 //          delta = softplus(dt + dt_bias); dt, A's row and D are indexed by c / ch_per_head, B and C by the group
@@ -39,7 +40,8 @@ causal_conv_silu_kernel(const T* __restrict__ rows, int row_elems, int col_off, 
                         const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
                         const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
                         const int* __restrict__ seq_first_row, const int* __restrict__ seq_start,
-                        const int* __restrict__ seq_end, T* __restrict__ out, int n_tok, int tokens_per_cta, int act) {
+                        const int* __restrict__ seq_end, T* __restrict__ out, int n_tok, int tokens_per_cta, int act,
+                        const float* __restrict__ in_bias) {
     grid_dependents_launch();
     grid_dependency_wait();
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -47,7 +49,7 @@ causal_conv_silu_kernel(const T* __restrict__ rows, int row_elems, int col_off, 
     float wk[16];
 #pragma unroll
     for (int j = 0; j < 16; ++j) wk[j] = j < K ? w[(size_t)c * K + K - 1 - j] : 0.f;      // wk[j]: the tap j tokens back
-    const float b = bias != nullptr ? bias[c] : 0.f;
+    const float b = bias != nullptr ? bias[c] : 0.f, xb = in_bias != nullptr ? in_bias[c] : 0.f;
     const int t_end = min(n_tok, ((int)blockIdx.x + 1) * tokens_per_cta);
     for (int t = blockIdx.x * tokens_per_cta; t < t_end; ++t) {
         const int s = tok_seq[t], slot = seq_slot[s], i = t - seq_first_row[s];
@@ -60,7 +62,7 @@ causal_conv_silu_kernel(const T* __restrict__ rows, int row_elems, int col_off, 
             if (j >= K) break;
             const int idx = i - j;
             float x = 0.f;
-            if (idx >= 0) x = to_float(rows[(size_t)(t - j) * row_elems + col_off + c]);
+            if (idx >= 0) x = to_float(rows[(size_t)(t - j) * row_elems + col_off + c]) + xb;
             else if (st != nullptr) x = st[(size_t)(K - 1 + idx) * C + c];
             xs[j] = x;
             acc = fmaf(wk[j], x, acc);
@@ -81,7 +83,8 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 conv_state_update_kernel(const T* __restrict__ rows, int row_elems, int col_off, int C, int K, float* __restrict__ state,
                          const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
-                         const int* __restrict__ seq_start, const int* __restrict__ seq_end) {
+                         const int* __restrict__ seq_start, const int* __restrict__ seq_end,
+                         const float* __restrict__ in_bias) {
     const int s = blockIdx.x;
     grid_dependents_launch();
     const int slot = seq_slot[s], row0 = seq_first_row[s], n = seq_end[s] - seq_start[s];
@@ -90,11 +93,12 @@ conv_state_update_kernel(const T* __restrict__ rows, int row_elems, int col_off,
     float* st = state + (size_t)slot * (K - 1) * C;
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
         float keep[15];
+        const float xb = in_bias != nullptr ? in_bias[c] : 0.f;
 #pragma unroll
         for (int jj = 0; jj < 15; ++jj) {
             if (jj >= K - 1) break;
             const int idx = n - (K - 1) + jj;
-            keep[jj] = idx >= 0 ? to_float(rows[(size_t)(row0 + idx) * row_elems + col_off + c]) : st[(size_t)(jj + n) * C + c];
+            keep[jj] = idx >= 0 ? to_float(rows[(size_t)(row0 + idx) * row_elems + col_off + c]) + xb : st[(size_t)(jj + n) * C + c];
         }
 #pragma unroll
         for (int jj = 0; jj < 15; ++jj) {
@@ -456,32 +460,32 @@ template <typename T>
 static int conv_launch(const void* rows, int row_elems, int col_off, int C, int K, const float* w, const float* bias,
                        float* state, const int* tok_seq, const int* seq_slot, const int* seq_first_row,
                        const int* seq_start, const int* seq_end, int n_tok, int n_seq, int one_token, void* out,
-                       int act, cudaStream_t stream) {
+                       int act, const float* in_bias, cudaStream_t stream) {
     const int by = (C + 255) / 256, tpc = n_tok >= 1024 ? 8 : 1;
     if (by > 65535) return fail("causal_conv_silu: too many channels (%d)", C);
     if (launch_kernel("causal_conv_silu", causal_conv_silu_kernel<T>, dim3((n_tok + tpc - 1) / tpc, by), dim3(256), 0, stream, 1,
                       (const T*)rows, row_elems, col_off, C, K, w, bias, state, tok_seq, seq_slot, seq_first_row, seq_start,
-                      seq_end, (T*)out, n_tok, tpc, act))
+                      seq_end, (T*)out, n_tok, tpc, act, in_bias))
         return 1;
     if (K <= 1 || one_token) return 0;
     return launch_kernel("conv_state_update", conv_state_update_kernel<T>, dim3(n_seq, by < 64 ? by : 64), dim3(256), 0, stream, 1,
-                         (const T*)rows, row_elems, col_off, C, K, state, seq_slot, seq_first_row, seq_start, seq_end);
+                         (const T*)rows, row_elems, col_off, C, K, state, seq_slot, seq_first_row, seq_start, seq_end, in_bias);
 }
 
 JANIS_EXPORT int janis_causal_conv_silu(const void* rows, int dtype, int row_elems, int col_off, int C, int K,
                                         const float* w, const float* bias, float* state, const int* tok_seq,
                                         const int* seq_slot, const int* seq_first_row, const int* seq_start,
                                         const int* seq_end, int n_tok, int n_seq, int one_token, void* out,
-                                        int act, cudaStream_t stream) {
+                                        int act, const float* in_bias, cudaStream_t stream) {
     if (n_tok <= 0 || n_seq <= 0) return 0;
     if (K < 1 || K > 16) return fail("causal_conv_silu: %d taps (1 to 16 are taken)", K);
     if (C <= 0 || col_off < 0 || col_off + C > row_elems) return fail("causal_conv_silu: channels %d at %d do not fit rows of %d", C, col_off, row_elems);
     if (dtype == JANIS_F32)
         return conv_launch<float>(rows, row_elems, col_off, C, K, w, bias, state, tok_seq, seq_slot, seq_first_row, seq_start,
-                                  seq_end, n_tok, n_seq, one_token, out, act, stream);
+                                  seq_end, n_tok, n_seq, one_token, out, act, in_bias, stream);
     if (dtype == JANIS_BF16)
         return conv_launch<bf16>(rows, row_elems, col_off, C, K, w, bias, state, tok_seq, seq_slot, seq_first_row, seq_start,
-                                 seq_end, n_tok, n_seq, one_token, out, act, stream);
+                                 seq_end, n_tok, n_seq, one_token, out, act, in_bias, stream);
     return fail("causal_conv_silu: unknown dtype %d", dtype);
 }
 
@@ -497,10 +501,10 @@ JANIS_EXPORT int janis_conv_state_update(const void* rows, int dtype, int row_el
     const dim3 grid(n_seq, by < 64 ? by : 64), block(256);
     if (dtype == JANIS_F32)
         return launch_kernel("conv_state_update", conv_state_update_kernel<float>, grid, block, 0, stream, 1, (const float*)rows,
-                             row_elems, col_off, C, K, state, seq_slot, seq_first_row, seq_start, seq_end);
+                             row_elems, col_off, C, K, state, seq_slot, seq_first_row, seq_start, seq_end, (const float*)nullptr);
     if (dtype == JANIS_BF16)
         return launch_kernel("conv_state_update", conv_state_update_kernel<bf16>, grid, block, 0, stream, 1, (const bf16*)rows,
-                             row_elems, col_off, C, K, state, seq_slot, seq_first_row, seq_start, seq_end);
+                             row_elems, col_off, C, K, state, seq_slot, seq_first_row, seq_start, seq_end, (const float*)nullptr);
     return fail("conv_state_update: unknown dtype %d", dtype);
 }
 

@@ -115,6 +115,7 @@ class DecoderModel:
         part.load(store, rt)
         for sub in part.sub_parts():
             self._load(sub, store, rt, done)
+        part.loaded(rt)
 
     def cache_line_needs(self) -> list[dict]:
         return [dict(self.blocks[self.schedule[self._writer[line]].layer].mixer.cache_needs())

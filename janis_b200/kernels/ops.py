@@ -23,9 +23,9 @@ PAGE = 64                      # tokens per cache page (JANIS_PAGE in the CUDA s
 GEMV_MAX_ROWS = 64             # what the skinny kernel accepts
 GEMV_FAST_ROWS = 16            # up to here it beats the library product (above, each warp re-reads too much of x)
 TC05_MAX_ROWS = 64             # rows the tcgen05 skinny product takes
-EPI_NONE, EPI_GATED_GELU, EPI_SOFTCAP, EPI_GATED_SILU = 0, 1, 2, 3
+EPI_NONE, EPI_GATED_GELU, EPI_SOFTCAP, EPI_GATED_SILU, EPI_GATED_CLAMP = 0, 1, 2, 3, 4
 GATE_GROUP = 8                 # fused gate/up rows alternate in groups of 8
-ACT_GELU_TANH, ACT_SILU = 0, 1
+ACT_GELU_TANH, ACT_SILU, ACT_CLAMPED = 0, 1, 2        # activations of a gated feed-forward (gated_act)
 
 _DT = {torch.float32: 0, torch.bfloat16: 1}
 
@@ -53,14 +53,14 @@ def core():
         lib.janis_embed.argtypes = [P, P, I, P, I, I, I, F, P]
         lib.janis_rmsnorm.argtypes = [P, I, P, P, P, I, I, I, F, P]
         lib.janis_add_rmsnorm.argtypes = [P, P, I, I, c_longlong, P, F, P, F, P, I, I, I, P]
-        lib.janis_gated_act.argtypes = [P, P, I, I, I, I, I, P]
+        lib.janis_gated_act.argtypes = [P, P, I, I, I, I, I, F, F, F, P]
         lib.janis_softcap.argtypes = [P, c_longlong, F, P]
         lib.janis_scale_values.argtypes = [P, c_longlong, F, P]
         lib.janis_bias_act.argtypes = [P, P, I, I, I, I, F, F, P]
         lib.janis_rope_store.argtypes = [P, I, P, P, P, P, P, I, I, I, I, I, I, P, P, P, I, I, I, P]
         lib.janis_kv_store.argtypes = [P, I, P, P, P, P, I, I, I, I, I, P, P, P, I, I, P]
         lib.janis_gemm_f32.argtypes = [P, P, P, I, I, I, F, P]
-        lib.janis_gemv_bf16.argtypes = [P, P, P, I, I, I, I, I, F, I, P]
+        lib.janis_gemv_bf16.argtypes = [P, P, P, I, I, I, I, I, F, I, F, F, P]
         lib.janis_gemv_bf16_bias_act.argtypes = [P, P, P, I, I, I, P, I, F, F, P]
         lib.janis_gemv_rope_store.argtypes = [P, P, P, I, I, P, P, P, P, P, I, I, I, I, P, P, P, I, I, P]
         lib.janis_gemm_tc05.argtypes = [P, P, P, I, I, I, I, I, F, I, P]
@@ -138,7 +138,7 @@ def mixers():
         _need_cuda()
         lib = build.mixers_library()
         P, I, F = c_void_p, c_int, c_float
-        lib.janis_qkv_rotate_store.argtypes = [P, I, I, P, P, P, P, I, P, I, I, I, I, I, I, P, P, P, I, P]
+        lib.janis_qkv_rotate_store.argtypes = [P, I, I, P, P, P, P, I, P, I, I, I, I, I, I, P, P, P, I, P, F, I, F, P, P]
         lib.janis_talk_attention.argtypes = [P, I, I, P, P, P, P, P, P, I, P, P, P, I, I, I, I, I, F, I, I, I, I, I, P, c_longlong, I, F, P, I, I, P, c_longlong, I, P]
         lib.janis_talk_attention_set_kernel.argtypes = [I]
         lib.janis_talk_attention_set_kernel.restype = None
@@ -148,12 +148,12 @@ def mixers():
         lib.janis_gla_scan.argtypes = [P, I, I, I, I, I, P, P, P, I, P, P, P, P, P, P, I, I, I, I, F, F, P]
         lib.janis_head_norm_gate.argtypes = [P, P, I, I, I, P, F, P, I, I, I, I, I, P]
         lib.janis_mlstm_scan.argtypes = [P, I, I, I, I, I, P, P, F, P, I, P, P, P, P, P, P, P, P, I, I, I, I, F, P]
-        lib.janis_causal_conv_silu.argtypes = [P, I, I, I, I, I, P, P, P, P, P, P, P, P, I, I, I, P, I, P]
+        lib.janis_causal_conv_silu.argtypes = [P, I, I, I, I, I, P, P, P, P, P, P, P, P, I, I, I, P, I, P, P]
         lib.janis_conv_state_update.argtypes = [P, I, I, I, I, I, P, P, P, P, P, I, P]
         lib.janis_qkv_conv_norm_store.argtypes = [P, I, I, I, I, I, I, I, I, P, P, P, P, I, F, P, P, P, P, P, P, P, P, P, P, I, P]
         lib.janis_latent_rotate_store.argtypes = [P, I, I, I, P, I, I, I, I, I, I, I, I, P, F, P, F, P, P, P, P, P, P, I, P]
         lib.janis_qk_rotate_norm_store.argtypes = [P, I, I, I, I, I, I, I, I, P, I, F, P, P, P, P, P, P, I, P]
-        lib.janis_head_linear.argtypes = [P, I, I, I, I, P, P, I, I, I, I, I, I, I, P]
+        lib.janis_head_linear.argtypes = [P, I, I, I, I, P, P, I, I, I, I, I, I, I, I, P]
         lib.janis_group_norm.argtypes = [P, P, I, P, F, P, F, I, P, I, I, I, P]
         lib.janis_round_rows.argtypes = [P, P, ctypes.c_size_t, P]
         lib.janis_selective_scan.argtypes = [P, I, I, I, P, I, I, P, P, I, P, I, I, I, P, P, I, I, P, P, P, P, I, P, P, I, I, I, I, I, P, P]
@@ -165,7 +165,11 @@ def mixers():
         lib.janis_dyt_norm.argtypes = [P, P, I, P, F, P, P, P, I, I, I, P]
         lib.janis_rmsnorm_accumulate.argtypes = [P, I, P, F, F, P, I, I, I, P]
         lib.janis_sigmoid_gate.argtypes = [P, P, I, I, I, I, I, I, P]
-        lib.janis_moe_route.argtypes = [P, P, I, I, I, I, I, F, I, P, I, I, P]
+        lib.janis_gate_place.argtypes = [P, P, I, I, I, I, P, I, I, F, I, I, P]
+        lib.janis_gated_recurrence_scan.argtypes = [P, I, P, c_longlong, c_longlong, P, P, P, P, I, I, P, P, P, P, P, I, P, P, I, I, F, I, I, P]
+        lib.janis_gated_recurrence_rows.argtypes = [P, I, P, P, P, P, P, I, I, P, P, P, I, P, P, I, I, F, I, I, P]
+        lib.janis_moe_relu2.argtypes = [P, I, P, I, I, I, I, I, I, P]
+        lib.janis_moe_route.argtypes = [P, P, I, I, I, I, I, F, I, P, I, I, I, P]
         lib.janis_moe_expert_act.argtypes = [P, I, P, I, I, F, I, F, F, P, I, I, F, P]
         lib.janis_moe_identity_add.argtypes = [P, P, I, P, I, I, I, I, P]
         lib.janis_hc_spread.argtypes = [P, P, I, I, I, P]
@@ -298,14 +302,16 @@ def add_rmsnorm(h, res, w_post, eps_post, w_next=None, eps_next=0.0, out=None, n
     return out
 
 
-def gated_act(gu, out, act: int = ACT_GELU_TANH, group: int = GATE_GROUP):
+def gated_act(gu, out, act: int = ACT_GELU_TANH, group: int = GATE_GROUP, limit: float = 0.0, alpha: float = 1.0,
+              up_add: float = 0.0):
     """out[r, j] = act(gate) * up over a fused [R, 2I] product whose columns alternate
-    `group` gate columns and `group` up columns."""
+    `group` gate columns and `group` up columns.  ACT_CLAMPED takes three numbers: g sigmoid(alpha g) (u + up_add) with
+    g = min(gate, limit), u = clamp(up, -limit, limit)."""
     R, I2 = gu.shape
     I = I2 // 2
     lib = core()
     _check(lib, lib.janis_gated_act(_t(gu, "gu", _FLOATS, (R, 2 * I)), _t(out, "out", gu.dtype, (R, I)),
-                                    _DT[gu.dtype], R, I, group, act, _stream()))
+                                    _DT[gu.dtype], R, I, group, act, float(limit), float(alpha), float(up_add), _stream()))
     return out
 
 
@@ -400,17 +406,22 @@ def gemm_f32(x, w, out, cap: float = 0.0):
     return out
 
 
-def gemv_bf16(x, w, out, epilogue: int = EPI_NONE, cap: float = 0.0, cluster: int = 0):
+_GATED = (EPI_GATED_GELU, EPI_GATED_SILU, EPI_GATED_CLAMP)
+
+
+def gemv_bf16(x, w, out, epilogue: int = EPI_NONE, cap: float = 0.0, cluster: int = 0, alpha: float = 1.0,
+              up_add: float = 0.0):
     """out = x[M<=64, K] w[N, K]^T, bfloat16 operands, float accumulation; out bfloat16 or float32
     [M, N], or [M, N/2] with a gated epilogue (rows of w alternate 8 gate rows and 8 up rows).
-    cluster: how many CTAs of a thread-block cluster share the K of a tile (1, 2, 4; 0 = chosen from N, K)."""
+    cluster: how many CTAs of a thread-block cluster share the K of a tile (1, 2, 4; 0 = chosen from N, K).
+    EPI_GATED_CLAMP: `cap` is the limit, alpha and up_add as in `gated_act`."""
     M, K = x.shape
     N = w.shape[0]
-    n_out = N // 2 if epilogue in (EPI_GATED_GELU, EPI_GATED_SILU) else N
+    n_out = N // 2 if epilogue in _GATED else N
     lib = core()
     _check(lib, lib.janis_gemv_bf16(_t(x, "x", torch.bfloat16, (M, K)), _t(w, "w", torch.bfloat16, (N, K)),
                                     _t(out, "out", _FLOATS, (M, n_out)), _DT[out.dtype], M, N, K, epilogue,
-                                    float(cap), int(cluster), _stream()))
+                                    float(cap), int(cluster), float(alpha), float(up_add), _stream()))
     return out
 
 
@@ -793,13 +804,18 @@ def attn_decode(qkv, kpool, vpool, page_table, seq_slot, seq_len, scratch, out, 
 # ---------------------------------------------------------------------------
 
 def qkv_rotate_store(rows, tok_pos, tok_seq, seq_slot, inv_qk, rot: int, inv_v, H: int, G: int, d: int, dv: int,
-                     kpool=None, vpool=None, page_table=None, store: bool = True):
+                     kpool=None, vpool=None, page_table=None, store: bool = True, bias=None, amplitude: float = 1.0,
+                     mix: int = 0, share: float = 0.0, v_first=None):
     """Rotary encoding of the first `rot` features of the queries and keys of a step (pairs i, i + rot/2), rotation
     of the values over all dv features by inv_v (None: values stay as projected), and the write of keys and values
     into the paged cache line.  rows [T, H d + G d + G dv] holds q, then k, then v; with store=False the rows hold q
-    alone.  kpool [pages, G, PAGE, d], vpool [pages, G, PAGE, dv]."""
+    alone.  kpool [pages, G, PAGE, d], vpool [pages, G, PAGE, dv].  bias (float32, one per column of q | k | v) is added
+    before anything else; `amplitude` multiplies sine and cosine of the queries' and keys' turn.  mix 1: the values are
+    also left in v_first [T, G dv]; mix 2: they become (1 - share) v + share v_first before they are stored."""
     T, width = rows.shape
     _t(rows, "rows", _FLOATS, (T, None))
+    if bias is not None and bias.numel() < H * d + (G * (d + dv) if store else 0):
+        raise KernelError("qkv_rotate_store: fewer biases than columns")
     if tok_pos.numel() < T or tok_seq.numel() < T:
         raise KernelError("qkv_rotate_store: position tables shorter than the step")
     _t(inv_qk, "inv_qk", torch.float32, (rot // 2,))
@@ -819,7 +835,8 @@ def qkv_rotate_store(rows, tok_pos, tok_seq, seq_slot, inv_qk, rot: int, inv_v, 
         seq_slot.data_ptr() if store else None, inv_qk.data_ptr() if rot else None, rot,
         inv_v.data_ptr() if inv_v is not None else None, T, H, G, d, dv, 1 if store else 0,
         kpool.data_ptr() if store else None, vpool.data_ptr() if store else None,
-        page_table.data_ptr() if store else None, stride, _stream()))
+        page_table.data_ptr() if store else None, stride, _t(bias, "bias", torch.float32) if bias is not None else None,
+        float(amplitude), int(mix), float(share), _t(v_first, "v_first", rows.dtype, (T, G * dv)) if mix else None, _stream()))
     return rows
 
 
@@ -1073,9 +1090,9 @@ def dyt_norm(h, res, alpha: float, weight, bias, out, rows=None):
 
 
 def causal_conv_silu(rows, col_off: int, channels: int, weight, bias, state, tok_seq, seq_slot, seq_first_row, seq_start,
-                     seq_end, n_seq: int, out, one_token: bool = False, act: bool = True):
+                     seq_end, n_seq: int, out, one_token: bool = False, act: bool = True, in_bias=None):
     """out[t, c] = silu(bias[c] + sum_j weight[c, K-1-j] x[t-j, c]) (act=False: without the silu; bias None: without
-    one) over the channels rows[:, col_off : col_off +
+    one; in_bias float32 [channels]: x is rows + in_bias, before the sequence's start still zero) over the channels rows[:, col_off : col_off +
     channels] of each sequence's tokens; inputs before the step come from state float32 [slots, max(K-1, 1), channels]
     (the last K-1 inputs of each slot), which is brought up to date: by the same kernel for sequences that bring one
     token, by a second kernel for the others (one_token=True: every sequence brings one, a decode step, and the
@@ -1097,7 +1114,9 @@ def causal_conv_silu(rows, col_off: int, channels: int, weight, bias, state, tok
                                            state.data_ptr(),
                                            tok_seq.data_ptr(), seq_slot.data_ptr(), seq_first_row.data_ptr(),
                                            seq_start.data_ptr(), seq_end.data_ptr(), T, n_seq, 1 if one_token else 0,
-                                           _t(out, "out", rows.dtype, (T, channels)), 1 if act else 0, _stream()),
+                                           _t(out, "out", rows.dtype, (T, channels)), 1 if act else 0,
+                                           _t(in_bias, "in_bias", torch.float32, (channels,)) if in_bias is not None else None,
+                                           _stream()),
            kernels=2 if K > 1 and not one_token else 1)
     return out
 
@@ -1196,6 +1215,73 @@ def sigmoid_gate(x, rows, g_off: int, per: int = 1):
     _check(lib, lib.janis_sigmoid_gate(_t(x, "x", _FLOATS, (T, n)), _t(rows, "rows", x.dtype, (T, None)), _DT[x.dtype],
                                        rows.shape[1], int(g_off), T, n, int(per), _stream()))
     return x
+
+
+def gate_place(x, rows, g_off: int, out, o_off: int = 0, scale: float = 1.0, per: int = 1):
+    """out[t, o_off + c] = scale * x[t, c] * sigmoid(rows[t, g_off + c // per]) (rows None: no gate): what `sigmoid_gate`
+    does, into columns of another tensor.  x [T, n], out [T, >= o_off + n] of x's dtype."""
+    T, n = x.shape
+    lib = mixers()
+    _check(lib, lib.janis_gate_place(_t(x, "x", _FLOATS, (T, n)), _t(rows, "rows", x.dtype, (T, None)) if rows is not None else None,
+                                     _DT[x.dtype], rows.shape[1] if rows is not None else 0, int(g_off), int(per),
+                                     _t(out, "out", x.dtype, (T, None)), out.shape[1], int(o_off), float(scale), T, n, _stream()))
+    return out
+
+
+def _recurrence_tables(name, T, C, u, bias_r, bias_i, decay, y_rows, y_off, y_bias, state, out, o_off):
+    _t(u, "u", _FLOATS, (T, C))
+    for n, v in (("bias_r", bias_r), ("bias_i", bias_i), ("decay", decay)) + ((("y_bias", y_bias),) if y_bias is not None else ()):
+        _t(v, n, torch.float32, (C,))
+    _t(y_rows, "y_rows", u.dtype, (T, None))
+    _t(state, "state", torch.float32, (None, C))
+    _t(out, "out", u.dtype, (T, None))
+    if y_off + C > y_rows.shape[1] or o_off + C > out.shape[1]:
+        raise KernelError(f"{name}: a column range lies outside its rows")
+
+
+def gated_recurrence_scan(u, gates, block: int, bias_r, bias_i, decay, y_rows, y_off: int, y_bias, seq_slot, seq_first_row,
+                          seq_start, seq_end, n_seq: int, state, out, o_off: int = 0, scale: float = 1.0):
+    """The gated linear recurrence over the tokens each sequence brings, in order: S <- a S + sqrt(1 - a^2) i u with
+    log a = decay sigmoid(zr + bias_r), i = sigmoid(zi + bias_i), and out[t, o_off + c] = scale S gelu_tanh(y + y_bias).
+    u [T, C]; gates float32 [T, C / block, 2 block]: zr of a block's channels, then zi; decay, biases float32 [C];
+    y = y_rows[:, y_off : y_off + C]; state float32 [slots, C], read and written back for slots >= 0."""
+    T, C = u.shape
+    _recurrence_tables("gated_recurrence_scan", T, C, u, bias_r, bias_i, decay, y_rows, y_off, y_bias, state, out, o_off)
+    _t(gates, "gates", torch.float32, (T, C // block, 2 * block))
+    for name, tab in (("seq_slot", seq_slot), ("seq_first_row", seq_first_row), ("seq_start", seq_start), ("seq_end", seq_end)):
+        _t(tab, name, torch.int32)
+        if tab.numel() < n_seq:
+            raise KernelError(f"gated_recurrence_scan: {name} shorter than the step's sequences")
+    lib = mixers()
+    _check(lib, lib.janis_gated_recurrence_scan(
+        u.data_ptr(), _DT[u.dtype], gates.data_ptr(), 2 * C, 2 * int(block), bias_r.data_ptr(), bias_i.data_ptr(), decay.data_ptr(),
+        y_rows.data_ptr(), y_rows.shape[1], int(y_off), y_bias.data_ptr() if y_bias is not None else None, seq_slot.data_ptr(),
+        seq_first_row.data_ptr(), seq_start.data_ptr(), seq_end.data_ptr(), n_seq, state.data_ptr(), out.data_ptr(), out.shape[1],
+        int(o_off), float(scale), C, int(block), _stream()))
+    return out
+
+
+REC_MAX_BLOCK = 1536       # channels a block of the recurrence's gates may have (its rows of u stand in shared memory)
+
+
+def gated_recurrence_rows(u, w, bias_r, bias_i, decay, y_rows, y_off: int, y_bias, tok_seq, seq_slot, state, out,
+                          o_off: int = 0, scale: float = 1.0):
+    """`gated_recurrence_scan` for a step whose sequences bring one token each, the gates' products included:
+    w [blocks, 2 block, block] holds a block's matrix of zr, then that of zi."""
+    T, C = u.shape
+    _recurrence_tables("gated_recurrence_rows", T, C, u, bias_r, bias_i, decay, y_rows, y_off, y_bias, state, out, o_off)
+    block = w.shape[2]
+    _t(w, "w", u.dtype, (C // block, 2 * block, block))
+    _t(tok_seq, "tok_seq", torch.int32)
+    _t(seq_slot, "seq_slot", torch.int32)
+    if tok_seq.numel() < T:
+        raise KernelError("gated_recurrence_rows: tok_seq shorter than the step")
+    lib = mixers()
+    _check(lib, lib.janis_gated_recurrence_rows(
+        u.data_ptr(), _DT[u.dtype], w.data_ptr(), bias_r.data_ptr(), bias_i.data_ptr(), decay.data_ptr(), y_rows.data_ptr(),
+        y_rows.shape[1], int(y_off), y_bias.data_ptr() if y_bias is not None else None, tok_seq.data_ptr(), seq_slot.data_ptr(),
+        T, state.data_ptr(), out.data_ptr(), out.shape[1], int(o_off), float(scale), C, block, _stream()))
+    return out
 
 
 def group_norm(h, res, alpha: float, weight, eps: float, groups: int, out, rows=None):
@@ -1322,13 +1408,13 @@ HEAD_LINEAR_FEW_ROWS = 64        # up to here the kernel that keeps its rows in 
 
 def head_linear(x, x_head: int, x_off: int, w, out, o_head: int, o_off: int):
     """out[t, h * o_head + o_off + o] = sum_i w[h, o, i] x[t, h * x_head + x_off + i]: a product per head with a
-    matrix of its own.  x [T, >= H x_head], w [H, O, I], out [T, >= H o_head], all of one dtype; float accumulation
-    (in float32, and for few rows, in an order that depends on I alone)."""
+    matrix of its own.  x [T, >= H x_head], w [H, O, I], out [T, >= H o_head], all of one dtype or out float32; float
+    accumulation (in float32, and for few rows, in an order that depends on I alone)."""
     T = x.shape[0]
     Hn, O, I = w.shape
     _t(x, "x", _FLOATS, (T, None))
     _t(w, "w", x.dtype, (Hn, O, I))
-    _t(out, "out", x.dtype, (T, None))
+    _t(out, "out", (x.dtype, torch.float32), (T, None))
     if (Hn - 1) * x_head + x_off + I > x.shape[1] or (Hn - 1) * o_head + o_off + O > out.shape[1]:
         raise KernelError("head_linear: the heads do not fit the rows")
     if x.dtype == torch.bfloat16 and T > HEAD_LINEAR_FEW_ROWS:
@@ -1336,32 +1422,37 @@ def head_linear(x, x_head: int, x_off: int, w, out, o_head: int, o_off: int):
         # `linear_bf16` takes the library product for its large cases
         xv = x.as_strided((Hn, T, I), (x_head, x.stride(0), 1), x.storage_offset() + x_off)
         ov = out.as_strided((Hn, T, O), (o_head, out.stride(0), 1), out.storage_offset() + o_off)
-        torch.bmm(xv, w.transpose(1, 2), out=ov)
+        if out.dtype == torch.float32:
+            torch.bmm(xv, w.transpose(1, 2), out_dtype=torch.float32, out=ov)
+        else:
+            torch.bmm(xv, w.transpose(1, 2), out=ov)
         return out
     lib = mixers()
     _check(lib, lib.janis_head_linear(x.data_ptr(), _DT[x.dtype], x.shape[1], int(x_head), int(x_off), w.data_ptr(),
-                                      out.data_ptr(), out.shape[1], int(o_head), int(o_off), T, Hn, I, O, _stream()))
+                                      out.data_ptr(), _DT[out.dtype], out.shape[1], int(o_head), int(o_off), T, Hn, I, O,
+                                      _stream()))
     return out
 
 
 def moe_route(z, correction, n_experts: int, group_count: int, group_keep: int, top: int, scale: float,
-              shared_gate: bool, out, n_identity: int = 0, softmax: bool = False):
+              shared_gate: bool, out, n_identity: int = 0, softmax: bool = False, group_best: bool = False):
     """The router's weights per token and expert, 0 for experts that were not chosen: s = sigmoid(z), choice scores
     s + correction, the best group_keep of group_count groups (by the sum of a group's two largest choice scores), the
     `top` largest choice scores among their experts, w = s / (sum of the chosen s + 1e-20) * scale.  With
     shared_gate, column n_experts of z is a gate's logit and column n_experts of out its sigmoid.  z, out float32.
     softmax: s = softmax(z) over all entries instead.  n_identity: that many more entries behind the experts in z and
     correction (before the gate's column); they are scored and chosen like experts, and the weights of the chosen ones
-    add up in one more column at the end of out."""
+    add up in one more column at the end of out.  group_best: a group's score is its largest choice score alone.
+    correction may be None (zeros)."""
     T = z.shape[0]
     n = n_experts + n_identity
     cols_in = n + (1 if shared_gate else 0)
     cols_out = n_experts + (1 if shared_gate else 0) + (1 if n_identity else 0)
     lib = mixers()
-    _check(lib, lib.janis_moe_route(_t(z, "z", torch.float32, (T, cols_in)), _t(correction, "correction", torch.float32, (n,)),
+    _check(lib, lib.janis_moe_route(_t(z, "z", torch.float32, (T, cols_in)), _t(correction, "correction", torch.float32, (n,)) if correction is not None else None,
                                     T, n_experts, int(group_count), int(group_keep), int(top), float(scale),
                                     1 if shared_gate else 0, _t(out, "out", torch.float32, (T, cols_out)), int(n_identity),
-                                    1 if softmax else 0, _stream()))
+                                    1 if softmax else 0, 1 if group_best else 0, _stream()))
     return out
 
 
@@ -1388,6 +1479,18 @@ def moe_expert_act(gu, wts, n_experts: int, ff: int, limit: float, shared_ff: in
                                          n_experts, ff, float(limit), int(shared_ff), float(shared_limit), float(alpha),
                                          _t(out, "out", gu.dtype, (T, total)), T, wts.shape[1], float(up_add), _stream()))
     return out
+
+
+def moe_relu2(x, wts, n_experts: int, ff: int, shared_ff: int = 0, shared_gate: bool = False):
+    """x[t, e * ff + j] = wts[t, e] * relu(x)^2 in place over the columns of all experts side by side; the shared expert's
+    shared_ff columns come last, with weight wts[t, E] (shared_gate) or 1."""
+    T, total = x.shape
+    if total != n_experts * ff + shared_ff:
+        raise KernelError(f"moe_relu2: rows of {total} for {n_experts} experts of {ff} and a shared one of {shared_ff}")
+    lib = mixers()
+    _check(lib, lib.janis_moe_relu2(_t(x, "x", _FLOATS, (T, total)), _DT[x.dtype], _t(wts, "wts", torch.float32, (T, None)),
+                                    wts.shape[1], n_experts, ff, int(shared_ff), 1 if shared_gate else 0, T, _stream()))
+    return x
 
 
 # ---------------------------------------------------------------------------

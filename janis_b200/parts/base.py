@@ -10,7 +10,8 @@ sequence after sequence without padding):
 
 * `Part.tensor_specs()` -> {checkpoint name: TensorSpec}: what it loads.
 * `Part.load(store, rt)`: take its tensors from the store (`store.get(name,
-  dtype)`), fuse or widen them as its kernels want.
+  dtype)`), fuse or widen them as its kernels want; `Part.loaded(rt)` comes once
+  its sub-parts have loaded too.
 * `Norm.forward(x, ctx, out, rows=None)`; `Norm.residual_add(h, r, ctx,
   next_norm=None, out=None)`: h += norm(r) on the float32 residual stream, and
   out = next_norm(h) when asked.
@@ -21,6 +22,13 @@ sequence after sequence without padding):
 * `Mixer.cache_needs()` -> {name: KVNeed | StateNeed}; `Mixer.forward(x, ctx,
   line)` -> [T, hidden] in the activation dtype.  `line[name]` is the cache part
   it asked for; `line.write` is False when the schedule lets it only read.
+* A mixer that begins with one product of its input and ends with one product
+  can share both with others that read the same input: it hands out
+  `in_weight()` [columns, hidden] and `out_weight()` [hidden, features] (and keeps
+  neither), and `join(rows, col0, ctx, line, z, z0, scale)` goes from its columns
+  of the shared product's rows to its features (times `scale`) in z's columns from
+  z0.  `joins`: "any", "first" (its columns must be the rows' first) or "" (it
+  cannot).
 * `FeedForward.forward(x, ctx)` -> [T, hidden].
 * `Block.forward(h, ctx, line, y_in=None, next_norm=None)` -> (h, y_next): h is the
   float32 residual stream, updated in place; y_in is this block's first norm
@@ -159,6 +167,9 @@ class Part:
     def load(self, store, rt: Runtime) -> None:
         pass
 
+    def loaded(self, rt: Runtime) -> None:
+        pass
+
     def sub_parts(self) -> list["Part"]:
         return []
 
@@ -194,6 +205,8 @@ class PositionEncoding(Part):
 
 
 class Mixer(Part):
+    joins = ""                      # "any", "first" or "": whether its products can be shared (see the module text)
+
     def cache_needs(self) -> Mapping[str, Any]:
         return {}
 
@@ -205,6 +218,15 @@ class Mixer(Part):
 
     def forward(self, x, ctx: StepContext, line):
         raise NotImplementedError
+
+    def in_weight(self):
+        raise NotImplementedError(f"{type(self).__name__} shares its products with no other mixer")
+
+    def out_weight(self):
+        raise NotImplementedError(f"{type(self).__name__} shares its products with no other mixer")
+
+    def join(self, rows, col0: int, ctx: StepContext, line, z, z0: int, scale: float) -> None:
+        raise NotImplementedError(f"{type(self).__name__} shares its products with no other mixer")
 
 
 class FeedForward(Part):

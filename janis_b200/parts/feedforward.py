@@ -4,7 +4,8 @@ down(act(up(x) + b_up)) + b_down (`DenseMLP`, at the end of the file).
 Gemma2's is GeGLU with the tanh form of gelu (`gemma/gemma.go:121-123`;
 0.5 v (1 + tanh(0.7978845608028654 (v + 0.044715 v^3))), `cpu/cpu.go:417-423`);
 with act="silu" it is the SwiGLU of the reference's other models
-(`qwen/mlp.go:32-36`).
+(`qwen/mlp.go:32-36`).  act="clamped_swish" is the gated form with limits:
+g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(alpha g) (u + 1).
 
 gate and up are one product: their rows are interleaved at load in groups of 8
 (8 gate rows, the 8 matching up rows, ...), which puts each gate value beside
@@ -21,20 +22,23 @@ import torch
 from ..weights.loader import TensorSpec
 from .base import FeedForward, Runtime, StepContext
 
-_ACTS = {"gelu_tanh": 0, "gelu_pytorch_tanh": 0, "silu": 1}
+_ACTS = {"gelu_tanh": 0, "gelu_pytorch_tanh": 0, "silu": 1, "clamped_swish": 2}
 
 
 class GatedMLP(FeedForward):
     GROUP = 8
 
     def __init__(self, hidden: int, intermediate: int, names: dict[str, str], act: str = "gelu_tanh",
-                 init_std: float = 0.02):
+                 init_std: float = 0.02, limit: float | None = None, gate_alpha: float = 1.702):
+        if act == "clamped_swish" and not (limit is not None and limit > 0):
+            raise ValueError(f"the clamped gate needs a positive limit, found {limit!r}")
         if act not in _ACTS:
             raise ValueError(f"unknown activation {act!r} (known: {sorted(_ACTS)})")
         for k in ("gate", "up", "down"):
             if k not in names:
                 raise ValueError(f"feed-forward needs the checkpoint name of its {k!r} projection")
         self.hidden, self.intermediate = hidden, intermediate
+        self.extra = {"limit": float(limit), "alpha": float(gate_alpha), "up_add": 1.0} if act == "clamped_swish" else {}
         # the fused gate/up layout wants whole groups: an intermediate width that is no multiple of the group is
         # padded with zero rows of gate and up (act(0) * 0 = 0) and zero columns of down
         self.padded = -(-intermediate // self.GROUP) * self.GROUP
@@ -70,15 +74,16 @@ class GatedMLP(FeedForward):
         rt, ws, ops = ctx.rt, ctx.ws, ctx.rt.ops
         T, I = ctx.n_tok, self.padded
         a = ws.buf("ffn.act", (T, I), rt.dtype)
-        epi = ops.EPI_GATED_GELU if self.act == 0 else ops.EPI_GATED_SILU
+        epi = (ops.EPI_GATED_GELU, ops.EPI_GATED_SILU, ops.EPI_GATED_CLAMP)[self.act]
         if rt.dtype == torch.bfloat16 and T <= ops.GEMV_FAST_ROWS and self.hidden % 8 == 0:   # (the skinny product reads 16 bytes at a time)
-            ops.gemv_bf16(x, self.w_gu, a, epi)
+            ops.gemv_bf16(x, self.w_gu, a, epi, **({"cap": self.extra["limit"], "alpha": self.extra["alpha"],
+                                                    "up_add": self.extra["up_add"]} if self.extra else {}))
         else:
             # (ops.gemm_tc05 computes this product with the activation fused for 17..64 rows, but at these
             # shapes the library product plus the activation kernel is still the faster pair)
             gu = ws.buf("ffn.gu", (T, 2 * I), rt.dtype)
             rt.linear(x, self.w_gu, gu)
-            ops.gated_act(gu, a, self.act, self.GROUP)
+            ops.gated_act(gu, a, self.act, self.GROUP, **self.extra)
         out = ws.buf("ffn.out", (T, self.hidden), rt.dtype)
         return rt.linear(a, self.w_down, out)
 

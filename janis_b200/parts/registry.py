@@ -43,6 +43,7 @@ def _register_builtin() -> None:
     from .embedding import Embedding, LMHead
     from .feedforward import DenseMLP, GatedMLP
     from .filtered_attention import FilteredAttention
+    from .gated_recurrence import GatedRecurrenceMixer
     from .hyper import HyperConnectionBlock, HyperRead
     from .matrix_memory import MatrixMemory
     from .latent_attention import LatentAttention
@@ -62,7 +63,8 @@ def _register_builtin() -> None:
     register("mixer", "matrix_memory", MatrixMemory)                      # a matrix, a normaliser and a running maximum per head, exponential gates
     register("mixer", "selective_scan", SelectiveScanMixer)               # a state per channel, step sizes through a low rank
     register("mixer", "state_space_duality", DualityMixer)                # a scalar decay per head, grouped B and C
-    register("mixer", "parallel", ParallelMixers)                         # branches on one input, normed and averaged
+    register("mixer", "gated_recurrence", GatedRecurrenceMixer)           # a number of state per channel, decays gated by the input
+    register("mixer", "parallel", ParallelMixers)                         # branches on one input, normed and averaged or added with constants
     register("feed_forward", "gated_mlp", GatedMLP)
     register("feed_forward", "dense_mlp", DenseMLP)                       # up, activation, down, with biases
     register("feed_forward", "routed_experts", RoutedExperts)             # a router over small gated experts, a shared one

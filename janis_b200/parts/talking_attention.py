@@ -22,7 +22,12 @@ projected, before any turn or norm (so the value size is the key size), cached b
 after the turn every head of q and k is divided by its own root mean square, sqrt(mean(head^2) + eps), without a
 weight.  A position encoding of pairs="neighbours" turns (2i, 2i + 1) instead of (i, i + rot/2).  `keep_first` (with
 a window): the sequence's first `keep_first` positions stay seen behind the window, at their true positions.
-`gate="head"`: Wg has one row per head and the gate is one number per head.
+`gate="head"`: Wg has one row per head and the gate is one number per head.  Biases on the projections (names
+["q_bias"], ["k_bias"], ["v_bias"], all three or none) are added before the turn.  A learnt sink (names["sink"], a number
+per head): exp(sink_h) joins the denominator instead of 1.  The position encoding's amplitude multiplies sine and cosine.
+`value_mix`: "first" leaves the layer's values where later layers of the step find them, "mix" makes the values
+(1 - m) v + m v_first with the stored number m (names["vmix"]) before they are cached, v_first being the values of the
+same token in the layer that left them.
 
 Keys and values live in a paged cache line with separate head sizes.  A step writes its keys and values first
 and then attends over the line alone, so a prompt, a prompt that continues, a decode step and a layer that reads
@@ -44,7 +49,7 @@ class TalkingHeadsAttention(Mixer):
                  position: RotaryEncoding, names: dict[str, str], value_position: RotaryEncoding | None = None,
                  block: int = 0, sink: bool = False, own_kv: bool = True, init_std: float = 0.02, window: int = 0,
                  keep_first: int = 0, values_from_keys: bool = False, unit_norm_eps: float | None = None,
-                 gate: str = "element"):
+                 gate: str = "element", value_mix: str | None = None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads do not divide over {n_kv_heads} key/value heads")
         if gate not in ("head", "element"):
@@ -57,6 +62,14 @@ class TalkingHeadsAttention(Mixer):
         self.values_from_keys = bool(values_from_keys)
         self.unit_norm_eps = None if unit_norm_eps is None else float(unit_norm_eps)
         self.gate = gate
+        if value_mix not in (None, "first", "mix") or (value_mix == "mix" and "vmix" not in names):
+            raise ValueError(f"value_mix is first or mix (with the checkpoint name of its number, 'vmix'), found {value_mix!r}")
+        biases = [b for b in ("q_bias", "k_bias", "v_bias") if b in names]
+        if biases and len(biases) != 3:
+            raise ValueError("biases stand on all three projections or on none")
+        if (biases or value_mix) and (not own_kv or values_from_keys or value_position is not None):
+            raise ValueError("biases and mixed values belong to a layer with plain values of its own")
+        self.value_mix, self.biased = value_mix, bool(biases)
         need = (("q", "k", "o") if values_from_keys else ("q", "k", "v", "o")) if own_kv else ("q", "o")
         for k in need:
             if k not in names:
@@ -70,12 +83,13 @@ class TalkingHeadsAttention(Mixer):
         self.window = int(window or 0)
         if self.window < 0:
             raise ValueError(f"a window holds at least one position, found {window}")
-        self.sink = bool(sink)
+        self.sink = bool(sink) or "sink" in names
         self.own_kv = bool(own_kv)
         self.position, self.value_position = position, value_position
         self.names = dict(names)
         self.init_std = init_std
-        self.w_qkv = self.w_o = self.talk = None
+        self.w_qkv = self.w_o = self.talk = self.bias = self.sink_values = None
+        self.mix_share = 0.0
 
     def tensor_specs(self):
         H, G, d, dv, W, s, n = self.n_heads, self.n_kv_heads, self.key_dim, self.value_dim, self.hidden, self.init_std, self.names
@@ -88,6 +102,13 @@ class TalkingHeadsAttention(Mixer):
             specs[n["talk"]] = TensorSpec((H, H), init_std=H ** -0.5)
         if "g" in n:
             specs[n["g"]] = TensorSpec((H * dv if self.gate == "element" else H, W), init_std=s)
+        if self.biased:
+            specs.update({n["q_bias"]: TensorSpec((H * d,), init_std=s), n["k_bias"]: TensorSpec((G * d,), init_std=s),
+                          n["v_bias"]: TensorSpec((G * dv,), init_std=s)})
+        if "sink" in n:
+            specs[n["sink"]] = TensorSpec((H,), init_std=1.0)
+        if self.value_mix == "mix":
+            specs[n["vmix"]] = TensorSpec((), init_std=0.1, init_mean=0.5)
         return specs
 
     def sub_parts(self):
@@ -126,49 +147,97 @@ class TalkingHeadsAttention(Mixer):
             pad = torch.zeros(8 - self.w_qkv.shape[0] % 8, self.w_qkv.shape[1], dtype=self.w_qkv.dtype, device=self.w_qkv.device)
             self.w_qkv = torch.cat([self.w_qkv, pad], dim=0).contiguous()
         self.w_o = store.get(n["o"], rt.dtype).contiguous()
+        f32 = lambda k: store.get(n[k]).to(torch.float32)
+        self.bias = torch.cat([f32("q_bias"), f32("k_bias"), f32("v_bias")]).contiguous() if self.biased else None
+        self.sink_values = f32("sink").contiguous() if "sink" in n else None
+        self.mix_share = float(f32("vmix").reshape(()).item()) if self.value_mix == "mix" else 0.0
         self.talk = store.get(n["talk"]).to(torch.float32).contiguous() if "talk" in n else None
 
+    @property
+    def joins(self):
+        return "first" if self.own_kv else ""
+
+    def in_weight(self):
+        w, self.w_qkv = self.w_qkv, None
+        return w
+
+    def out_weight(self):
+        w, self.w_o = self.w_o, None
+        return w
+
+    def _gate_off(self) -> int:                     # where the gate's logits start in a row
+        H, G, d, dv = self.n_heads, self.n_kv_heads, self.key_dim, self.value_dim
+        return H * d + ((G * d if self.values_from_keys else G * (d + dv)) if self.own_kv else 0)
+
+    def _gate_run(self) -> int:                     # features that share a gate
+        return self.value_dim if self.gate == "head" else 1
+
     def forward(self, x, ctx: StepContext, line):
+        rt, ws, ops = ctx.rt, ctx.ws, ctx.rt.ops
+        T = ctx.n_tok
+        rows = ws.buf("tattn.rows", (T, self.w_qkv.shape[0]), rt.dtype)      # (the product's columns: the gate's, and padding, last)
+        rt.linear(x, self.w_qkv, rows)
+        att = self._attend(rows, ctx, line)
+        if "g" in self.names:
+            ops.sigmoid_gate(att, rows, self._gate_off(), per=self._gate_run())
+        return rt.linear(att, self.w_o, ws.buf("mixer.out", (T, self.hidden), rt.dtype))
+
+    def join(self, rows, col0: int, ctx: StepContext, line, z, z0: int, scale: float) -> None:
+        if col0:
+            raise ValueError("an attention's columns are the first of the rows it shares")
+        att = self._attend(rows, ctx, line)
+        ctx.rt.ops.gate_place(att, rows if "g" in self.names else None, self._gate_off(), z, z0, scale, per=self._gate_run())
+
+    def _attend(self, rows, ctx: StepContext, line):
+        """From the projected rows (q | k | v first) to the heads side by side, [T, H dv]; keys and values are stored."""
         rt, ws, ops = ctx.rt, ctx.ws, ctx.rt.ops
         kv = line["kv"]
         if kv.write != self.own_kv:
             raise ValueError("the schedule lets a layer with keys and values of its own only read a line, or the reverse")
         T, H, G, d, dv = ctx.n_tok, self.n_heads, self.n_kv_heads, self.key_dim, self.value_dim
-        kv_cols = (G * d if self.values_from_keys else G * (d + dv)) if self.own_kv else 0
-        g_off = H * d + kv_cols                                        # where the gate's logits start in a row
-        rows = ws.buf("tattn.rows", (T, self.w_qkv.shape[0]), rt.dtype)      # (the product's columns: the gate's, and padding, last)
-        rt.linear(x, self.w_qkv, rows)
         inv_v = self.value_position.inv_freq if self.value_position is not None else None
         neighbours = self.position.pairs == "neighbours" and self.position.rot > 0
         if self.values_from_keys or self.unit_norm_eps is not None or neighbours:
-            if inv_v is not None or not self.own_kv or self.position.amplitude != 1.0:
-                raise NotImplementedError("turned values, a borrowed line or an amplitude together with normed or neighbouring pairs")
+            if inv_v is not None or not self.own_kv or self.position.amplitude != 1.0 or self.biased or self.value_mix:
+                raise NotImplementedError("turned or mixed values, biases, a borrowed line or an amplitude together with normed or neighbouring pairs")
             if not self.values_from_keys:
                 raise NotImplementedError("normed or neighbouring pairs beside a value projection of its own")
             ops.qk_rotate_norm_store(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, self.position.inv_freq, self.position.rot,
                                      not neighbours, self.unit_norm_eps is not None, self.unit_norm_eps or 0.0, H, G, d,
                                      kv.k, kv.v if self.values_from_keys else None, kv.table)
         else:
+            extras = {}
+            if self.biased:
+                extras["bias"] = self.bias
+            if self.position.amplitude != 1.0:
+                extras["amplitude"] = self.position.amplitude
+            if self.value_mix == "first":           # (the step's later layers read it: a buffer of its own)
+                extras.update(mix=1, v_first=ws.buf("tattn.v_first", (T, G * dv), rt.dtype))
+                ctx.shared["first values"] = extras["v_first"]
+            elif self.value_mix == "mix":
+                extras.update(mix=2, share=self.mix_share, v_first=ctx.shared["first values"])
             ops.qkv_rotate_store(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, self.position.inv_freq, self.position.rot,
                                  inv_v, H, G, d, dv, kv.k if self.own_kv else None, kv.v if self.own_kv else None,
-                                 kv.table if self.own_kv else None, store=self.own_kv)
+                                 kv.table if self.own_kv else None, store=self.own_kv, **extras)
         att = ws.buf("tattn.ctx", (T, H * dv), rt.dtype)
+        more = {}
+        if self.keep_first:
+            more["keep_first"] = self.keep_first
+        if self.sink_values is not None:
+            more["sink_values"] = self.sink_values
         decode = ctx.mode == "decode"
         max_keys, n_chunks, scratch = 0, 1, None
         rows_floats = 0
-        if (decode and rt.dtype == torch.bfloat16 and not self.block and not self.sink and self.talk is None and inv_v is None
-                and hasattr(ops, "talk_attention_rows_floats")):
+        if (decode and rt.dtype == torch.bfloat16 and not self.block and self.talk is None and inv_v is None
+                and (not self.sink or self.sink_values is not None) and hasattr(ops, "talk_attention_rows_floats")):
             # a decode step in the serving dtype with nothing the kernels that take single rows leave out: keys and
             # values read once, 16 bytes a lane
             max_keys = min(ctx.len_bound, self.window + self.keep_first) if self.window else ctx.len_bound
             rows_floats = ops.talk_attention_rows_floats(rt.dtype, T, H, G, d, dv, max_keys)
         if rows_floats:
-            ops.talk_attention_rows(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, kv.k, kv.v, kv.table, None, att, H, G, d, dv,
-                                    self.scale, ws.buf("tattn.rows_scratch", (rows_floats,), torch.float32), max_keys,
-                                    window=self.window, **({"keep_first": self.keep_first} if self.keep_first else {}))
-            if "g" in self.names:
-                ops.sigmoid_gate(att, rows, g_off, per=dv if self.gate == "head" else 1)
-            return rt.linear(att, self.w_o, ws.buf("mixer.out", (T, self.hidden), rt.dtype))
+            return ops.talk_attention_rows(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, kv.k, kv.v, kv.table, None, att, H, G, d, dv,
+                                           self.scale, ws.buf("tattn.rows_scratch", (rows_floats,), torch.float32), max_keys,
+                                           sink=self.sink, window=self.window, **more)
         if decode:
             # a decode row's keys over several CTAs when the rows alone would leave most of the GPU idle: about a
             # CTA an SM in all, none with fewer than 128 keys (the bound on the lengths is the host's)
@@ -178,10 +247,6 @@ class TalkingHeadsAttention(Mixer):
             n_chunks = max(1, min(rt.sm_count // max(T, 1), -(-max_keys // 128), 64))
             n = ops.talk_attention_scratch_floats(T, n_chunks, H, dv)
             scratch = ws.buf("tattn.partial", (n,), torch.float32) if n else None
-        ops.talk_attention(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, kv.k, kv.v, kv.table, self.talk, inv_v, att,
-                           H, G, d, dv, self.scale, self.block, self.sink, one_row=decode, max_keys=max_keys,
-                           n_chunks=n_chunks, scratch=scratch, window=self.window,
-                           **({"keep_first": self.keep_first} if self.keep_first else {}))
-        if "g" in self.names:
-            ops.sigmoid_gate(att, rows, g_off, per=dv if self.gate == "head" else 1)
-        return rt.linear(att, self.w_o, ws.buf("mixer.out", (T, self.hidden), rt.dtype))
+        return ops.talk_attention(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, kv.k, kv.v, kv.table, self.talk, inv_v, att,
+                                  H, G, d, dv, self.scale, self.block, self.sink, one_row=decode, max_keys=max_keys,
+                                  n_chunks=n_chunks, scratch=scratch, window=self.window, **more)

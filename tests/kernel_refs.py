@@ -15,9 +15,9 @@ import torch
 PAGE = 64
 GEMV_MAX_ROWS = 64
 GEMV_FAST_ROWS = 16
-EPI_NONE, EPI_GATED_GELU, EPI_SOFTCAP, EPI_GATED_SILU = 0, 1, 2, 3
+EPI_NONE, EPI_GATED_GELU, EPI_SOFTCAP, EPI_GATED_SILU, EPI_GATED_CLAMP = 0, 1, 2, 3, 4
 GATE_GROUP = 8
-ACT_GELU_TANH, ACT_SILU = 0, 1
+ACT_GELU_TANH, ACT_SILU, ACT_CLAMPED = 0, 1, 2
 
 
 def embed(tokens, table, scale, out):
@@ -53,10 +53,18 @@ def _act(g, act):
     return g / (1.0 + torch.exp(-g))
 
 
-def gated_act(gu, out, act=ACT_GELU_TANH, group=GATE_GROUP):
+def _clamped(gate, up, limit, alpha, up_add):
+    g = torch.clamp(gate, max=limit)
+    return g * torch.sigmoid(alpha * g) * (torch.clamp(up, min=-limit, max=limit) + up_add)
+
+
+def gated_act(gu, out, act=ACT_GELU_TANH, group=GATE_GROUP, limit=0.0, alpha=1.0, up_add=0.0):
     R, I2 = gu.shape
     I = I2 // 2
     v = gu.double().view(R, I // group, 2, group)
+    if act == ACT_CLAMPED:
+        out.copy_(_clamped(v[:, :, 0], v[:, :, 1], limit, alpha, up_add).reshape(R, I).to(out.dtype))
+        return out
     out.copy_((_act(v[:, :, 0], act) * v[:, :, 1]).reshape(R, I).to(out.dtype))
     return out
 
@@ -115,8 +123,12 @@ def gemm_f32(x, w, out, cap=0.0):
     return out
 
 
-def gemv_bf16(x, w, out, epilogue=EPI_NONE, cap=0.0, cluster=0):
+def gemv_bf16(x, w, out, epilogue=EPI_NONE, cap=0.0, cluster=0, alpha=1.0, up_add=0.0):
     v = x.double() @ w.double().T
+    if epilogue == EPI_GATED_CLAMP:
+        g = v.view(v.shape[0], v.shape[1] // 16, 2, 8)
+        out.copy_(_clamped(g[:, :, 0], g[:, :, 1], cap, alpha, up_add).reshape(v.shape[0], -1).to(out.dtype))
+        return out
     if epilogue in (EPI_GATED_GELU, EPI_GATED_SILU):
         M, N = v.shape
         g = v.view(M, N // 16, 2, 8)
@@ -332,18 +344,30 @@ def _turn(x, pos, inv, sign=1.0):
 
 
 def qkv_rotate_store(rows, tok_pos, tok_seq, seq_slot, inv_qk, rot, inv_v, H, G, d, dv, kpool=None, vpool=None,
-                     page_table=None, store=True):
+                     page_table=None, store=True, bias=None, amplitude=1.0, mix=0, share=0.0, v_first=None):
     T = rows.shape[0]
     for t in range(T):
         pos = int(tok_pos[t])
         n = H + G if store else H
         qk = rows[t, :n * d].view(n, d)
-        qk.copy_(_turn(qk, pos, inv_qk).to(rows.dtype))
+        x = qk.double()
+        if bias is not None:
+            x = x + bias[:n * d].double().view(n, d)
+        y = _turn(x, pos, inv_qk)
+        y[:, :2 * inv_qk.numel()] *= float(np.float32(amplitude))
+        qk.copy_(y.to(rows.dtype))
         if not store:
             continue
         v = rows[t, n * d:n * d + G * dv].view(G, dv)
         if inv_v is not None:
             v.copy_(_turn(v, pos, inv_v).to(rows.dtype))
+        if bias is not None or mix:
+            x = v.double() + (bias[n * d:n * d + G * dv].double().view(G, dv) if bias is not None else 0.0)
+            if mix == 2:
+                x = (1.0 - share) * x + share * v_first[t].double().view(G, dv)
+            v.copy_(x.to(rows.dtype))
+            if mix == 1:
+                v_first[t] = v.reshape(-1)
         slot = int(seq_slot[int(tok_seq[t])])
         if slot < 0:
             continue
@@ -455,7 +479,7 @@ def dyt_norm(h, res, alpha, weight, bias, out, rows=None):
 
 
 def causal_conv_silu(rows, col_off, channels, weight, bias, state, tok_seq, seq_slot, seq_first_row, seq_start, seq_end,
-                     n_seq, out, one_token=False, act=True):
+                     n_seq, out, one_token=False, act=True, in_bias=None):
     taps = weight.shape[1]
     w, b = weight.double(), bias.double() if bias is not None else torch.zeros(channels, dtype=torch.float64)
     for s in range(n_seq):
@@ -463,6 +487,8 @@ def causal_conv_silu(rows, col_off, channels, weight, bias, state, tok_seq, seq_
         if n <= 0:
             continue
         x = rows[row0:row0 + n, col_off:col_off + channels].double()
+        if in_bias is not None:
+            x = x + in_bias.double()
         past = state[slot, :taps - 1].double() if slot >= 0 else torch.zeros(taps - 1, channels, dtype=torch.float64)
         full = torch.cat([past, x], dim=0)                                  # local index i lives at i + taps - 1
         acc = b.expand(n, channels).clone()
@@ -638,16 +664,17 @@ def head_linear(x, x_head, x_off, w, out, o_head, o_off):
     return out
 
 
-def moe_route(z, correction, n_experts, group_count, group_keep, top, scale, shared_gate, out, n_identity=0, softmax=False):
+def moe_route(z, correction, n_experts, group_count, group_keep, top, scale, shared_gate, out, n_identity=0, softmax=False,
+              group_best=False):
     T = z.shape[0]
     real = n_experts
     n_experts = real + n_identity          # the entries that are scored and chosen
     s = torch.softmax(z[:, :n_experts].double(), -1) if softmax else torch.sigmoid(z[:, :n_experts].double())
-    c = s + correction.double()
+    c = s + correction.double() if correction is not None else s
     per = n_experts // group_count
     out.zero_()
     for t in range(T):
-        gs = [sum(sorted(c[t, g * per:(g + 1) * per].tolist(), reverse=True)[:2]) for g in range(group_count)]
+        gs = [sum(sorted(c[t, g * per:(g + 1) * per].tolist(), reverse=True)[:1 if group_best else 2]) for g in range(group_count)]
         kept = sorted(range(group_count), key=lambda g: (-gs[g], g))[:group_keep]
         cand = [e for g in sorted(kept) for e in range(g * per, (g + 1) * per)]
         chosen = sorted(cand, key=lambda e: (-float(c[t, e]), e))[:top]
@@ -779,3 +806,59 @@ def mlstm_scan(rows, q_off, k_off, v_off, z, bias, cap, seq_slot, seq_first_row,
             state_n[slot] = nn.float()[:, None, :].expand(H, state_n.shape[2], d)
             state_m[slot] = m.float()
     return o_out
+
+
+# ---------------------------------------------------------------------------
+# a gate on the way into a shared output product, experts of one matrix up, the gated linear recurrence
+# ---------------------------------------------------------------------------
+
+def gate_place(x, rows, g_off, out, o_off=0, scale=1.0, per=1):
+    v = x.double()
+    if rows is not None:
+        v = v * torch.sigmoid(rows[:, g_off:g_off + x.shape[1] // per].double().repeat_interleave(per, dim=1))
+    out[:, o_off:o_off + x.shape[1]] = (scale * v).to(out.dtype)
+    return out
+
+
+def moe_relu2(x, wts, n_experts, ff, shared_ff=0, shared_gate=False):
+    w = wts[:, :n_experts].double().repeat_interleave(ff, dim=1)
+    if shared_ff:
+        sw = wts[:, n_experts:n_experts + 1].double() if shared_gate else torch.ones(x.shape[0], 1, dtype=torch.float64)
+        w = torch.cat([w, sw.expand(-1, shared_ff)], dim=1)
+    x.copy_((w * torch.clamp(x.double(), min=0.0) ** 2).to(x.dtype))
+    return x
+
+
+def gated_recurrence_scan(u, gates, block, bias_r, bias_i, decay, y_rows, y_off, y_bias, seq_slot, seq_first_row, seq_start,
+                          seq_end, n_seq, state, out, o_off=0, scale=1.0):
+    T, C = u.shape
+    z = gates.double().view(T, C // block, 2, block)
+    r = torch.sigmoid(z[:, :, 0].reshape(T, C) + bias_r.double())
+    i = torch.sigmoid(z[:, :, 1].reshape(T, C) + bias_i.double())
+    y = y_rows[:, y_off:y_off + C].double() + (y_bias.double() if y_bias is not None else 0.0)
+    branch = _act(y, ACT_GELU_TANH)
+    for s in range(n_seq):
+        slot, row0, n = int(seq_slot[s]), int(seq_first_row[s]), int(seq_end[s]) - int(seq_start[s])
+        if n <= 0:
+            continue
+        S = state[slot].double().clone() if slot >= 0 else torch.zeros(C, dtype=torch.float64)
+        for t in range(row0, row0 + n):
+            la = decay.double() * r[t]
+            S = torch.exp(la) * S + torch.sqrt(-torch.expm1(2.0 * la)) * i[t] * u[t].double()
+            out[t, o_off:o_off + C] = (scale * S * branch[t]).to(out.dtype)
+        if slot >= 0:
+            state[slot] = S.float()
+    return out
+
+
+REC_MAX_BLOCK = 1536
+
+
+def gated_recurrence_rows(u, w, bias_r, bias_i, decay, y_rows, y_off, y_bias, tok_seq, seq_slot, state, out, o_off=0, scale=1.0):
+    T, C = u.shape
+    block = w.shape[2]
+    gates = torch.einsum("tbi,boi->tbo", u.double().view(T, C // block, block), w.double())
+    rows = torch.arange(T, dtype=torch.int32)
+    slots = torch.tensor([int(seq_slot[int(tok_seq[t])]) for t in range(T)], dtype=torch.int32)
+    return gated_recurrence_scan(u, gates, block, bias_r, bias_i, decay, y_rows, y_off, y_bias, slots, rows,
+                                 torch.zeros_like(rows), torch.ones_like(rows), T, state, out, o_off, scale)

@@ -569,15 +569,82 @@ def dekutar_like(gemma: dict, layers: int) -> dict:
             "norm": {"eps": 1e-6}, "logit_scale": 1.0, "layers": out}
 
 
+def larulorn_like(gemma: dict, layers: int) -> dict:
+    """A Larulorn configuration with the layer sizes of a Gemma2 one: the same width, heads, head size (for keys and
+    values), feed-forward width and vocabulary; layers alternate "parallel" (gated attention beside a gated linear recurrence
+    as wide as the model, a block of gates per head) and "attention" (biases, a sink per head, half the head turned, values
+    mixed from the first such layer); feed-forwards as `nosolix_like` has them: dense, dense, then mixtures of 16 experts, 4
+    chosen from the best 2 of 4 groups, with a shared expert; the plain experts have one matrix up instead of two, so they
+    are half as wide again: as many active feed-forward weights a token as the dense layer."""
+    hd, W, ff = int(gemma["head_dim"]), int(gemma["hidden_size"]), int(gemma["intermediate_size"])
+    H, G = gemma["num_attention_heads"], gemma["num_key_value_heads"]
+    base = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5}
+    left = dict(base, rot={"base": 10000.0, "dims": hd})
+    att = dict(base, v_mix=True, rot={"base": 10000.0, "dims": hd // 2,
+                                      "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}})
+    right = {"width": W, "blocks": max(b for b in range(1, H + 1) if W % b == 0), "conv": 4}
+    e_ff = max(8, ff * 3 // 8 // 8 * 8)
+    moe = {"kind": "moe", "expert": {"ff": e_ff}, "shared": {"ff": e_ff},
+           "router": {"experts": 16, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    out = []
+    for i in range(layers):
+        mixer = copy.deepcopy(att) if i % 2 else {"left": copy.deepcopy(left), "right": dict(right), "left_scale": 0.5, "right_scale": 0.5}
+        mlp = {"kind": "dense", "ff": ff, "limit": 7.0} if i % 4 < 2 else copy.deepcopy(moe)
+        out.append({"type": "attention" if i % 2 else "parallel", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Larulorn", "vocab": gemma["vocab_size"], "width": W, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "layers": out}
+
+
 _TIMED = {"sigalorn": ("talk_attention", "qkv_rotate_store", "gla_scan", "head_norm_gate", "bias_act", "add_rmsnorm", "rmsnorm"),
           "gemma2": ("attn_prefill", "attn_decode", "rope_store", "gemv_rope_store", "gated_act"),
-          "nosolix": ("talk_attention", "qkv_rotate_store", "selective_scan", "causal_conv_silu", "gate_group_norm",
+          "nosolix": ("talk_attention", "talk_attention_rows", "qkv_rotate_store", "selective_scan", "causal_conv_silu", "gate_group_norm",
                       "moe_route", "moe_expert_act", "dyt_norm", "rmsnorm_accumulate", "sigmoid_gate", "bias_act"),
           "dekutar": ("talk_attention", "talk_attention_rows", "qk_rotate_norm_store", "latent_rotate_store", "head_linear", "mlstm_scan",
                       "head_norm_gate", "hc_update", "hc_read_norm", "hc_spread", "sigmoid_gate", "moe_route", "moe_expert_act",
                       "moe_identity_add", "rmsnorm"),
+          "larulorn": ("talk_attention", "talk_attention_rows", "qkv_rotate_store", "causal_conv_silu", "head_linear",
+                       "gated_recurrence_scan", "gated_recurrence_rows", "gate_place", "moe_route", "moe_relu2", "gated_act",
+                       "add_rmsnorm", "rmsnorm"),
           "vivazen": ("talk_attention", "talk_attention_rows", "qkv_conv_norm_store", "latent_rotate_store", "head_linear", "group_norm", "round_rows",
                       "sigmoid_gate", "gated_act")}
+
+
+def _plain_kernel_bytes(model, rows: int) -> dict:
+    """Bytes that the kernels between a design's products must move in a step of `rows` tokens in bfloat16, by name: every
+    input read once, every output written once (the recurrence: its inputs, its output and its float32 gates)."""
+    from .parts.feedforward import DenseMLP, GatedMLP
+    from .parts.gated_recurrence import GatedRecurrenceMixer
+    from .parts.moe import RoutedExperts
+    from .parts.state_space import DualityMixer, SelectiveScanMixer
+    out: dict = {}
+
+    def add(name, per_row):
+        out[name] = out.get(name, 0) + rows * per_row
+
+    for call in model.schedule:
+        block = model.blocks[call.layer]
+        for m in _leaf_mixers(block.mixer):
+            joined = getattr(block.mixer, "scales", None) is not None
+            if isinstance(m, GatedRecurrenceMixer):
+                add("causal_conv_silu", 4 * m.width)
+                add("gated_recurrence_scan", (2 + 8 + 2 + 2) * m.width)                 # u, two float logits, the branch, the result
+            elif isinstance(m, SelectiveScanMixer):
+                add("causal_conv_silu", 4 * m.inner)
+                add("selective_scan", (2 + 2 + 2 + 2) * m.inner + 4 * m.state)           # u, dt, z, the result; B and C
+            elif isinstance(m, DualityMixer):
+                add("causal_conv_silu", 4 * m.conv_channels)
+                add("selective_scan", (2 + 4) * m.inner + 2 * m.n_heads + 4 * m.groups * m.state)
+                add("gate_group_norm", (4 + 2 + 2) * m.inner)
+            if "g" in getattr(m, "names", {}) and hasattr(m, "value_dim") and hasattr(m, "n_heads"):
+                add("gate_place" if joined else "sigmoid_gate", 6 * m.n_heads * m.value_dim)
+        f = getattr(block, "feed_forward", None)
+        if isinstance(f, RoutedExperts):
+            add("moe_relu2" if f.act == "relu2" else "moe_expert_act", (4 if f.act == "relu2" else 6) * f.total_ff)
+        elif isinstance(f, GatedMLP):
+            add("gated_act", 6 * f.padded)
+        elif isinstance(f, DenseMLP):
+            add("bias_act", 4 * f.intermediate)
+    return out
 
 
 def _leaf_mixers(mixer):
@@ -638,13 +705,16 @@ def _measure_design(raw: dict, kind: str, pk: dict, prefill_tokens: int, batch: 
                 elif isinstance(need, StateNeed) and name in ("state", "memory"):      # (a convolution's kept inputs are another kernel's)
                     gla_flops += mixer.prompt_flops(prefill_tokens)
                     state_bytes += 2 * batch * int(np.prod(need.shape)) * 4
+                    if kind == "larulorn":       # the kernel of single rows also reads the gates' matrices
+                        state_bytes += mixer.w_gates.numel() * mixer.w_gates.element_size()
                 elif isinstance(need, StateNeed) and name in ("normaliser", "maximum"):   # the matrix memory's other parts
                     state_bytes += 2 * batch * int(np.prod(need.shape)) * 4
     att_name = "attn_prefill" if kind == "gemma2" else "talk_attention"
     dec_name = "attn_decode" if kind == "gemma2" else "talk_attention"
     if kernels["decode_us"].get("talk_attention_rows"):      # decode steps through the kernels that take single rows
         dec_name = "talk_attention_rows"
-    scan_name = {"nosolix": "selective_scan", "dekutar": "mlstm_scan"}.get(kind, "gla_scan")
+    scan_name = {"nosolix": "selective_scan", "dekutar": "mlstm_scan", "larulorn": "gated_recurrence_scan"}.get(kind, "gla_scan")
+    scan_decode = "gated_recurrence_rows" if kind == "larulorn" else scan_name
     roof = {}
     if kernels["prefill_us"].get(att_name):
         roof["attention_prefill_frac_of_bf16_peak"] = round(att_flops / (kernels["prefill_us"][att_name] * 1e-6) / (pk["bf16_tflops"] * 1e12), 5)
@@ -653,10 +723,18 @@ def _measure_design(raw: dict, kind: str, pk: dict, prefill_tokens: int, batch: 
         dec_us = (kernels["decode_us"].get("talk_attention") or 0.0) + (kernels["decode_us"].get("talk_attention_rows") or 0.0)
     if dec_us:
         roof["attention_decode_frac_of_copy_bandwidth"] = round(kv_bytes / (dec_us * 1e-6) / 1e9 / pk["hbm_gbs"], 5)
-    if kernels["prefill_us"].get(scan_name):
+    if kernels["prefill_us"].get(scan_name) and kind != "larulorn":      # (whose recurrence is bound by its bytes: below)
         roof["recurrence_prefill_tflops_fp32"] = round(gla_flops / (kernels["prefill_us"][scan_name] * 1e-6) / 1e12, 3)
-    if kernels["decode_us"].get(scan_name):
-        roof["recurrence_decode_frac_of_copy_bandwidth"] = round(state_bytes / (kernels["decode_us"][scan_name] * 1e-6) / 1e9 / pk["hbm_gbs"], 5)
+    if kernels["decode_us"].get(scan_decode):
+        roof["recurrence_decode_frac_of_copy_bandwidth"] = round(state_bytes / (kernels["decode_us"][scan_decode] * 1e-6) / 1e9 / pk["hbm_gbs"], 5)
+    if kind in ("nosolix", "larulorn"):
+        for nm, nbytes in _plain_kernel_bytes(model, prefill_tokens).items():
+            if kernels["prefill_us"].get(nm):
+                roof[f"{nm}_prefill_frac_of_copy_bandwidth"] = round(nbytes / (kernels["prefill_us"][nm] * 1e-6) / 1e9 / pk["hbm_gbs"], 5)
+        if kernels["prefill_us"].get("head_linear") and kind == "larulorn":
+            fl = sum(4.0 * m.width * m.width // m.blocks * prefill_tokens for c in model.schedule for m in _leaf_mixers(model.blocks[c.layer].mixer)
+                     if hasattr(m, "w_gates") and hasattr(m, "blocks"))
+            roof["head_linear_prefill_frac_of_bf16_peak"] = round(fl / (kernels["prefill_us"]["head_linear"] * 1e-6) / (pk["bf16_tflops"] * 1e12), 5)
     # the elementwise kernels of a step against the bytes of the residual stream they pass over (one float32 read and
     # write and one activation written per norm): the norms' share, a number to set beside the other design's
     T = prefill_tokens
@@ -697,7 +775,8 @@ def compare(sizes=("gemma2-2b", "gemma2-9b", "gemma2-27b"), layers: int = 4, pre
     weights: prompt tokens a second, decode tokens a second, and the device time of each design's own kernels in
     one prompt step and one decode step with what fraction of the roofline that is."""
     pk, pk_kind = peaks()
-    rec = {"compare": f"{design} beside {'sigalorn' if design in ('nosolix', 'vivazen', 'dekutar') else 'gemma2'}", "dtype": "bf16", "data": "synthetic",
+    beside = {"larulorn": "nosolix", "sigalorn": "gemma2"}.get(design, "sigalorn")
+    rec = {"compare": f"{design} beside {beside}", "dtype": "bf16", "data": "synthetic",
            "peaks": pk_kind, "prefill_tokens": prefill_tokens, "batch": batch, "context": context, "steps": steps, "sizes": {}}
     for name in sizes:
         gemma = dict(load_config(name), num_hidden_layers=layers)
@@ -711,6 +790,11 @@ def compare(sizes=("gemma2-2b", "gemma2-9b", "gemma2-27b"), layers: int = 4, pre
             rec["sizes"][name] = {
                 "sigalorn": _measure_design(sigalorn_like(gemma, layers), "sigalorn", pk, prefill_tokens, batch, context, steps, warmup),
                 "dekutar": _measure_design(dekutar_like(gemma, layers), "dekutar", pk, prefill_tokens, batch, context, steps, warmup)}
+            continue
+        if design == "larulorn":     # beside the design it is closest to: attention beside a recurrence, dense layers and routed experts
+            rec["sizes"][name] = {
+                "nosolix": _measure_design(nosolix_like(gemma, layers), "nosolix", pk, prefill_tokens, batch, context, steps, warmup),
+                "larulorn": _measure_design(larulorn_like(gemma, layers), "larulorn", pk, prefill_tokens, batch, context, steps, warmup)}
             continue
         if design == "nosolix":      # beside the closest design the library has: recurrent layers between attention over a limited span
             rec["sizes"][name] = {
@@ -744,9 +828,9 @@ def main(argv=None) -> int:
                     "instead of sequences that all reach --context")
     ap.add_argument("--profile", choices=["decode", "prefill"], default="",
                     help="open the CUDA profiler range around two timed decode steps, or the last prompt step")
-    ap.add_argument("--compare", choices=["sigalorn", "nosolix", "vivazen", "dekutar"], default="",
-                    help="instead of the benchmark: Sigalorn beside Gemma2, or Nosolix, Vivazen or Dekutar beside Sigalorn, at equal layer "
-                    "sizes (prompt and decode throughput, and each design's own kernels against their rooflines); "
+    ap.add_argument("--compare", choices=["sigalorn", "nosolix", "vivazen", "dekutar", "larulorn"], default="",
+                    help="instead of the benchmark: Sigalorn beside Gemma2, Nosolix, Vivazen or Dekutar beside Sigalorn, or Larulorn beside "
+                    "Nosolix, at equal layer sizes (prompt and decode throughput, and each design's own kernels against their rooflines); "
                     "--config picks one size")
     a = ap.parse_args(argv)
     if a.impl == "reference":

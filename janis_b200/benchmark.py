@@ -597,12 +597,12 @@ def larulorn_like(gemma: dict, layers: int) -> dict:
 
 _TIMED = {"sigalorn": ("talk_attention", "qkv_rotate_store", "gla_scan", "head_norm_gate", "bias_act", "add_rmsnorm", "rmsnorm"),
           "gemma2": ("attn_prefill", "attn_decode", "rope_store", "gemv_rope_store", "gated_act"),
-          "nosolix": ("talk_attention", "talk_attention_rows", "qkv_rotate_store", "selective_scan", "causal_conv_silu", "gate_group_norm",
+          "nosolix": ("talk_attention", "talk_attention_rows", "attn_prefill_rows", "attn_decode_rows", "qkv_rotate_store", "selective_scan", "causal_conv_silu", "gate_group_norm",
                       "moe_route", "moe_expert_act", "dyt_norm", "rmsnorm_accumulate", "sigmoid_gate", "bias_act"),
           "dekutar": ("talk_attention", "talk_attention_rows", "qk_rotate_norm_store", "latent_rotate_store", "head_linear", "mlstm_scan",
                       "head_norm_gate", "hc_update", "hc_read_norm", "hc_spread", "sigmoid_gate", "moe_route", "moe_expert_act",
                       "moe_identity_add", "rmsnorm"),
-          "larulorn": ("talk_attention", "talk_attention_rows", "qkv_rotate_store", "causal_conv_silu", "head_linear",
+          "larulorn": ("talk_attention", "talk_attention_rows", "attn_prefill_rows", "attn_decode_rows", "qkv_rotate_store", "causal_conv_silu", "head_linear",
                        "gated_recurrence_scan", "gated_recurrence_rows", "gate_place", "moe_route", "moe_relu2", "gated_act",
                        "add_rmsnorm", "rmsnorm"),
           "vivazen": ("talk_attention", "talk_attention_rows", "qkv_conv_norm_store", "latent_rotate_store", "head_linear", "group_norm", "round_rows",
@@ -713,6 +713,10 @@ def _measure_design(raw: dict, kind: str, pk: dict, prefill_tokens: int, batch: 
     dec_name = "attn_decode" if kind == "gemma2" else "talk_attention"
     if kernels["decode_us"].get("talk_attention_rows"):      # decode steps through the kernels that take single rows
         dec_name = "talk_attention_rows"
+    if kernels["prefill_us"].get("attn_prefill_rows"):       # attention through the kernels of whole heads
+        att_name = "attn_prefill_rows"
+    if kernels["decode_us"].get("attn_decode_rows"):
+        dec_name = "attn_decode_rows"
     scan_name = {"nosolix": "selective_scan", "dekutar": "mlstm_scan", "larulorn": "gated_recurrence_scan"}.get(kind, "gla_scan")
     scan_decode = "gated_recurrence_rows" if kind == "larulorn" else scan_name
     roof = {}

@@ -257,7 +257,7 @@ __global__ void __launch_bounds__(ATTN_WARPS * 32)
 attn_decode_kernel(const T* __restrict__ qkv, const T* __restrict__ kpool, const T* __restrict__ vpool,
                    const int* __restrict__ page_table, int table_stride, const int* __restrict__ seq_slot,
                    const int* __restrict__ seq_len, float* __restrict__ partial, int nq, int nkv,
-                   int q_row_heads, float scale, float cap, int window, int ring_len, int chunk) {
+                   int q_stride, float scale, float cap, int window, int ring_len, int chunk) {
     typedef Geo<T> G;
     __shared__ float sm[ATTN_WARPS][G::RG][HD + 2];
     const int s = blockIdx.z;
@@ -282,7 +282,7 @@ attn_decode_kernel(const T* __restrict__ qkv, const T* __restrict__ kpool, const
 
     Lane<T> st;
     st.init();
-    const T* qrow = qkv + (size_t)s * q_row_heads * HD;
+    const T* qrow = qkv + (size_t)s * q_stride;
 #pragma unroll
     for (int r = 0; r < G::RG; ++r) st.load_q(qrow + (size_t)(h0 + r) * HD, r, r < nh_here, scale, lig);
 
@@ -401,7 +401,7 @@ __global__ void __launch_bounds__(Staged<T>::WARPS * 32)
 attn_decode_staged_kernel(const T* __restrict__ qkv, const T* __restrict__ kpool, const T* __restrict__ vpool,
                           const int* __restrict__ page_table, int table_stride, const int* __restrict__ seq_slot,
                           const int* __restrict__ seq_len, float* __restrict__ partial, int nq, int nkv,
-                          int q_row_heads, float scale, float cap, int window, int ring_len, int chunk) {
+                          int q_stride, float scale, float cap, int window, int ring_len, int chunk) {
     typedef Staged<T> S;
     typedef Geo<T, S::LMAX, S::BUDGET> G;
     extern __shared__ __align__(128) unsigned char stage_mem[];
@@ -455,7 +455,7 @@ attn_decode_staged_kernel(const T* __restrict__ qkv, const T* __restrict__ kpool
 
     Lane<T, S::LMAX, S::BUDGET> st;
     st.init();
-    const T* qrow = qkv + (size_t)s * q_row_heads * HD;
+    const T* qrow = qkv + (size_t)s * q_stride;
 #pragma unroll
     for (int r = 0; r < G::RG; ++r) st.load_q(qrow + (size_t)(h0 + r) * HD, r, r < nh_here, scale, lig);
 
@@ -541,8 +541,9 @@ template <int RB, bool DIRECT, int NS, bool WIDE = false>
 __global__ void __launch_bounds__(MmaDecode<NS, WIDE>::WARPS * 32)
 attn_decode_mma_kernel(const bf16* __restrict__ qkv, const bf16* __restrict__ kpool, const bf16* __restrict__ vpool,
                        const int* __restrict__ page_table, int table_stride, const int* __restrict__ seq_slot,
-                       const int* __restrict__ seq_len, float* __restrict__ partial, int nq, int nkv, int q_row_heads,
-                       float scale, float cap, int window, int ring_len, int chunk, bf16* __restrict__ out) {
+                       const int* __restrict__ seq_len, float* __restrict__ partial, int nq, int nkv, int q_stride,
+                       float scale, float cap, int window, int ring_len, int chunk, bf16* __restrict__ out,
+                       const float* __restrict__ sinks) {
     typedef MmaDecode<NS, WIDE> S;
     extern __shared__ __align__(128) unsigned char stage_mem[];
     __shared__ __align__(8) unsigned long long full[S::STAGES];
@@ -641,7 +642,7 @@ attn_decode_mma_kernel(const bf16* __restrict__ qkv, const bf16* __restrict__ kp
     // each block of 32 features, the 8 features t*8 .. t*8+7 as the pairs that two k-steps want
     uint32_t qf[S::KB][4];
     {
-        const bf16* qrow = qkv + (size_t)s * q_row_heads * HD + (size_t)(h0 + g) * HD;
+        const bf16* qrow = qkv + (size_t)s * q_stride + (size_t)(h0 + g) * HD;
 #pragma unroll
         for (int kb = 0; kb < S::KB; ++kb) {
             uint4 v = make_uint4(0, 0, 0, 0);
@@ -799,6 +800,7 @@ attn_decode_mma_kernel(const bf16* __restrict__ qkv, const bf16* __restrict__ kp
                     l += sm[w][r][1] * e;
                 }
             }
+            if (sinks != nullptr) l += expf(sinks[h0 + r] - mx);
             out[((size_t)s * nq + h0 + r) * HD + d] = __float2bfloat16_rn(v / l);
         }
     } else {
@@ -822,12 +824,13 @@ attn_decode_mma_kernel(const bf16* __restrict__ qkv, const bf16* __restrict__ kp
     }
 }
 
-// Merge of the chunks in ascending order.  One CTA per (sequence, head): the chunks' weights
+// Merge of the chunks in ascending order (with `sinks`, exp of head h's number joins its denominator: a key of that score
+// without a value).  One CTA per (sequence, head): the chunks' weights
 // exp(m_c - m) / l are formed once in shared memory, then each thread sums its features.
 template <typename T>
 __global__ void attn_merge_kernel(const float* __restrict__ partial, const int* __restrict__ seq_slot,
                                   const int* __restrict__ seq_len, T* __restrict__ out, int nq, int max_chunks,
-                                  int window, int chunk) {
+                                  int window, int chunk, const float* __restrict__ sinks) {
     extern __shared__ float wgt[];            // max_chunks weights
     __shared__ float red[32];
     const int s = blockIdx.x, h = blockIdx.y;
@@ -857,6 +860,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ partial, const int* 
         const float w = mc == -INFINITY ? 0.f : expf(mc - mx);
         float l = 0.f;                           // in chunk order, the same in every thread
         for (int c = 0; c < n_chunks; ++c) l += __shfl_sync(0xffffffffu, lc * w, c);
+        if (sinks != nullptr) l += expf(sinks[h] - mx);
         const float inv = 1.0f / l;
         for (int d0 = 0; d0 < HD; d0 += blockDim.x) {         // the same trips for every lane: the shuffles stay whole
             const int d = d0 + threadIdx.x;
@@ -889,6 +893,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ partial, const int* 
         float l = 0.f;                           // in chunk order, the same in every thread
         for (int c = 0; c < 32; ++c) l += __shfl_sync(0xffffffffu, lc0 * w_lo, c);
         for (int c = 32; c < n_chunks; ++c) l += __shfl_sync(0xffffffffu, lc1 * w_hi, c - 32);
+        if (sinks != nullptr) l += expf(sinks[h] - mx);
         const float inv = 1.0f / l;
         for (int d0 = 0; d0 < HD; d0 += blockDim.x) {
             const int d = d0 + threadIdx.x;
@@ -925,6 +930,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ partial, const int* 
     __syncthreads();
     float l = 0.f;                               // in chunk order, the same in every thread
     for (int c = 0; c < n_chunks; ++c) l += p[(size_t)c * (HD + 2) + 1] * wgt[c];
+    if (sinks != nullptr) l += expf(sinks[h] - mx);
     const float inv = 1.0f / l;
     for (int d = threadIdx.x; d < HD; d += blockDim.x) {
         float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;     // four running sums keep four loads in flight
@@ -1025,8 +1031,8 @@ JANIS_EXPORT int janis_attn_wait_probe(int tries, int* status, cudaStream_t stre
 template <int RB, int NS, bool WIDE = false>
 static int launch_decode_mma_ns(const bf16* qkv, const bf16* kpool, const bf16* vpool, const int* page_table,
                                 int table_stride, const int* seq_slot, const int* seq_len, float* partial, int n_seq, int nq,
-                                int nkv, int q_row_heads, float scale, float cap, int window, int ring_len, int chunk,
-                                int max_chunks, bf16* out, cudaStream_t stream) {
+                                int nkv, int q_stride, float scale, float cap, int window, int ring_len, int chunk,
+                                int max_chunks, bf16* out, const float* sinks, cudaStream_t stream) {
     typedef MmaDecode<NS, WIDE> S;
     static bool configured = false;
     if (!configured) {
@@ -1044,10 +1050,10 @@ static int launch_decode_mma_ns(const bf16* qkv, const bf16* kpool, const bf16* 
     if (out != nullptr)
         return launch_kernel("attn_decode", attn_decode_mma_kernel<RB, true, NS, WIDE>, grid, dim3(S::WARPS * 32),
                              S::SMEM_BYTES, stream, 1, qkv, kpool, vpool, page_table, table_stride, seq_slot, seq_len,
-                             partial, nq, nkv, q_row_heads, scale, cap, window, ring_len, chunk, out);
+                             partial, nq, nkv, q_stride, scale, cap, window, ring_len, chunk, out, sinks);
     return launch_kernel("attn_decode", attn_decode_mma_kernel<RB, false, NS, WIDE>, grid, dim3(S::WARPS * 32),
                          S::SMEM_BYTES, stream, 1, qkv, kpool, vpool, page_table, table_stride, seq_slot, seq_len,
-                         partial, nq, nkv, q_row_heads, scale, cap, window, ring_len, chunk, out);
+                         partial, nq, nkv, q_stride, scale, cap, window, ring_len, chunk, out, sinks);
 }
 
 static int decode_sm_count() {
@@ -1078,28 +1084,28 @@ JANIS_EXPORT int janis_attn_decode_stages(long long n_ctas) {
 template <int RB>
 static int launch_decode_mma_rb(const bf16* qkv, const bf16* kpool, const bf16* vpool, const int* page_table,
                                 int table_stride, const int* seq_slot, const int* seq_len, float* partial, int n_seq, int nq,
-                                int nkv, int q_row_heads, float scale, float cap, int window, int ring_len, int chunk,
-                                int max_chunks, bf16* out, cudaStream_t stream) {
+                                int nkv, int q_stride, float scale, float cap, int window, int ring_len, int chunk,
+                                int max_chunks, bf16* out, const float* sinks, cudaStream_t stream) {
     const int rep = nq / nkv;
     const long long n_ctas = (long long)max_chunks * nkv * ((rep + RB - 1) / RB) * n_seq;
     if (HD > 128 && g_mma_wide && n_ctas <= decode_sm_count())       // a CTA an SM at most: stages of 64 keys
         return launch_decode_mma_ns<RB, 2, true>(qkv, kpool, vpool, page_table, table_stride, seq_slot, seq_len, partial, n_seq, nq,
-                                                 nkv, q_row_heads, scale, cap, window, ring_len, chunk, max_chunks, out, stream);
+                                                 nkv, q_stride, scale, cap, window, ring_len, chunk, max_chunks, out, sinks, stream);
     if (janis_attn_decode_stages(n_ctas) == 2)
         return launch_decode_mma_ns<RB, 2>(qkv, kpool, vpool, page_table, table_stride, seq_slot, seq_len, partial, n_seq, nq, nkv,
-                                           q_row_heads, scale, cap, window, ring_len, chunk, max_chunks, out, stream);
+                                           q_stride, scale, cap, window, ring_len, chunk, max_chunks, out, sinks, stream);
     return launch_decode_mma_ns<RB, 3>(qkv, kpool, vpool, page_table, table_stride, seq_slot, seq_len, partial, n_seq, nq, nkv,
-                                       q_row_heads, scale, cap, window, ring_len, chunk, max_chunks, out, stream);
+                                       q_stride, scale, cap, window, ring_len, chunk, max_chunks, out, sinks, stream);
 }
 
 static int launch_decode_mma(const bf16* qkv, const bf16* kpool, const bf16* vpool, const int* page_table, int table_stride,
                              const int* seq_slot, const int* seq_len, float* partial, int n_seq, int nq, int nkv,
-                             int q_row_heads, float scale, float cap, int window, int ring_len, int chunk, int max_chunks,
-                             bf16* out, cudaStream_t stream) {
+                             int q_stride, float scale, float cap, int window, int ring_len, int chunk, int max_chunks,
+                             bf16* out, const float* sinks, cudaStream_t stream) {
     const int rep = nq / nkv;
 #define JANIS_RB(RB)                                                                                                   \
     return launch_decode_mma_rb<RB>(qkv, kpool, vpool, page_table, table_stride, seq_slot, seq_len, partial, n_seq, nq, nkv, \
-                                    q_row_heads, scale, cap, window, ring_len, chunk, max_chunks, out, stream)
+                                    q_stride, scale, cap, window, ring_len, chunk, max_chunks, out, sinks, stream)
     if (rep == 1) JANIS_RB(1);
     if (rep == 2) JANIS_RB(2);
     if (rep <= 4) JANIS_RB(4);
@@ -1110,15 +1116,15 @@ static int launch_decode_mma(const bf16* qkv, const bf16* kpool, const bf16* vpo
 template <typename T>
 static int launch_decode(const T* qkv, const T* kpool, const T* vpool, const int* page_table, int table_stride,
                          const int* seq_slot, const int* seq_len, float* partial, T* out, int n_seq, int nq, int nkv,
-                         int q_row_heads, float scale, float cap, int window, int ring_len, int chunk, int max_chunks,
-                         cudaStream_t stream) {
+                         int q_stride, float scale, float cap, int window, int ring_len, int chunk, int max_chunks,
+                         const float* sinks, cudaStream_t stream) {
     const int rep = nq / nkv;
     if (g_decode_kernel == 2 && sizeof(T) == 2 && MmaDecode<2>::OK) {
         // a launch of one chunk per sequence writes the result itself: no partials, no merge
         bf16* direct = max_chunks == 1 ? (bf16*)out : nullptr;
         if (launch_decode_mma((const bf16*)qkv, (const bf16*)kpool, (const bf16*)vpool, page_table, table_stride, seq_slot,
-                              seq_len, partial, n_seq, nq, nkv, q_row_heads, scale, cap, window, ring_len, chunk, max_chunks,
-                              direct, stream))
+                              seq_len, partial, n_seq, nq, nkv, q_stride, scale, cap, window, ring_len, chunk, max_chunks,
+                              direct, sinks, stream))
             return 1;
         if (direct != nullptr) return 0;
     } else if (g_decode_kernel >= 1) {
@@ -1134,26 +1140,29 @@ static int launch_decode(const T* qkv, const T* kpool, const T* vpool, const int
         }
         if (launch_kernel("attn_decode", attn_decode_staged_kernel<T>, grid, dim3(Staged<T>::WARPS * 32), Staged<T>::SMEM_BYTES,
                           stream, 1, qkv, kpool, vpool, page_table, table_stride, seq_slot, seq_len, partial, nq, nkv,
-                          q_row_heads, scale, cap, window, ring_len, chunk))
+                          q_stride, scale, cap, window, ring_len, chunk))
             return 1;
     } else {
         dim3 grid(max_chunks, nkv * ((rep + Geo<T>::RG - 1) / Geo<T>::RG), n_seq);
         if (launch_kernel("attn_decode", attn_decode_kernel<T>, grid, dim3(ATTN_WARPS * 32), 0, stream, 1, qkv, kpool, vpool,
-                          page_table, table_stride, seq_slot, seq_len, partial, nq, nkv, q_row_heads, scale, cap, window,
+                          page_table, table_stride, seq_slot, seq_len, partial, nq, nkv, q_stride, scale, cap, window,
                           ring_len, chunk))
             return 1;
     }
     dim3 mgrid(n_seq, nq);
     const int mthreads = HD < 256 ? (HD < 32 ? 32 : HD) : 256;
     return launch_kernel("attn_merge", attn_merge_kernel<T>, mgrid, dim3(mthreads), max_chunks * sizeof(float), stream, 1,
-                         (const float*)partial, seq_slot, seq_len, out, nq, max_chunks, window, chunk);
+                         (const float*)partial, seq_slot, seq_len, out, nq, max_chunks, window, chunk, sinks);
 }
 
-JANIS_EXPORT int janis_attn_decode(const void* qkv, const void* kpool, const void* vpool, int dtype,
-                                   const int* page_table, int table_stride, const int* seq_slot,
-                                   const int* seq_len, float* partial, long long partial_floats, void* out,
-                                   int n_seq, int nq, int nkv, int q_row_heads, float scale, float cap, int window,
-                                   int ring_len, int chunk, int max_chunks, cudaStream_t stream) {
+// janis_attn_decode with rows of q_stride elements between neighbouring queries and, when `sinks` ([nq] floats) is given,
+// exp(sinks[h]) in head h's denominator.
+JANIS_EXPORT int janis_attn_decode_sinks(const void* qkv, const void* kpool, const void* vpool, int dtype,
+                                         const int* page_table, int table_stride, const int* seq_slot,
+                                         const int* seq_len, float* partial, long long partial_floats, void* out,
+                                         int n_seq, int nq, int nkv, int q_stride, float scale, float cap, int window,
+                                         int ring_len, int chunk, int max_chunks, const float* sinks,
+                                         cudaStream_t stream) {
     if (n_seq <= 0) return 0;
     if (nkv <= 0 || nq % nkv) return fail("attn_decode: %d query heads do not divide over %d key heads", nq, nkv);
     if (chunk <= 0 || chunk % JANIS_PAGE) return fail("attn_decode: chunk %d is not a multiple of the page", chunk);
@@ -1161,6 +1170,7 @@ JANIS_EXPORT int janis_attn_decode(const void* qkv, const void* kpool, const voi
     if (ring_len > 0 && (window <= 0 || window > ring_len))
         return fail("attn_decode: window %d does not fit its ring of %d", window, ring_len);
     if (max_chunks <= 0) return fail("attn_decode: max_chunks must be positive");
+    if (q_stride < nq * HD || q_stride % 8) return fail("attn_decode: rows of %d elements for %d heads of %d", q_stride, nq, HD);
     if (partial_floats < janis_attn_decode_scratch(n_seq, nq, max_chunks))
         return fail("attn_decode: scratch of %lld floats is too small, %lld needed", partial_floats,
                     janis_attn_decode_scratch(n_seq, nq, max_chunks));
@@ -1168,13 +1178,23 @@ JANIS_EXPORT int janis_attn_decode(const void* qkv, const void* kpool, const voi
     if (max_chunks > 8192) return fail("attn_decode: too many chunks (%d)", max_chunks);
     if (dtype == JANIS_F32)
         return launch_decode<float>((const float*)qkv, (const float*)kpool, (const float*)vpool, page_table, table_stride,
-                                    seq_slot, seq_len, partial, (float*)out, n_seq, nq, nkv, q_row_heads, scale, cap,
-                                    window, ring_len, chunk, max_chunks, stream);
+                                    seq_slot, seq_len, partial, (float*)out, n_seq, nq, nkv, q_stride, scale, cap,
+                                    window, ring_len, chunk, max_chunks, sinks, stream);
     if (dtype == JANIS_BF16)
         return launch_decode<bf16>((const bf16*)qkv, (const bf16*)kpool, (const bf16*)vpool, page_table, table_stride,
-                                   seq_slot, seq_len, partial, (bf16*)out, n_seq, nq, nkv, q_row_heads, scale, cap,
-                                   window, ring_len, chunk, max_chunks, stream);
+                                   seq_slot, seq_len, partial, (bf16*)out, n_seq, nq, nkv, q_stride, scale, cap,
+                                   window, ring_len, chunk, max_chunks, sinks, stream);
     return fail("attn_decode: unknown dtype %d", dtype);
+}
+
+JANIS_EXPORT int janis_attn_decode(const void* qkv, const void* kpool, const void* vpool, int dtype,
+                                   const int* page_table, int table_stride, const int* seq_slot,
+                                   const int* seq_len, float* partial, long long partial_floats, void* out,
+                                   int n_seq, int nq, int nkv, int q_row_heads, float scale, float cap, int window,
+                                   int ring_len, int chunk, int max_chunks, cudaStream_t stream) {
+    return janis_attn_decode_sinks(qkv, kpool, vpool, dtype, page_table, table_stride, seq_slot, seq_len, partial,
+                                   partial_floats, out, n_seq, nq, nkv, q_row_heads * HD, scale, cap, window, ring_len,
+                                   chunk, max_chunks, nullptr, stream);
 }
 
 JANIS_EXPORT const char* janis_last_error() { return error_buffer(); }

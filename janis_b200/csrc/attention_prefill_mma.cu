@@ -106,9 +106,9 @@ template <bool EXT>
 __global__ void __launch_bounds__(THREADS)
 attn_prefill_mma_kernel(const bf16* __restrict__ q_src, const bf16* __restrict__ kv_src,
                         const int* __restrict__ seq_first_row, const int* __restrict__ seq_len, int n_seq,
-                        bf16* __restrict__ out, int nq, int nkv, int q_row_heads, int kv_row_heads,
+                        bf16* __restrict__ out, int nq, int nkv, int q_row_elems, int kv_row_elems,
                         int kv_k_head0, float scale, float cap, int window, int parts, int piece,
-                        float* __restrict__ partial, CachedPrefix cached) {
+                        float* __restrict__ partial, CachedPrefix cached, const float* __restrict__ sinks) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
     // Which sequence, which tile of BM queries and which part of its keys is this CTA's.  Items are handed
     // out from the end of the list: the last tiles of a sequence see the most keys and should start first.
@@ -133,7 +133,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q_src, const bf16* __restrict__
     const uint32_t sQ = (uint32_t)__cvta_generic_to_shared(smem_raw);
     const uint32_t sKV = sQ + Q_BYTES;                // stage s: K at sKV + s * 2 KV_BYTES, V right after
 
-    const size_t q_stride = (size_t)q_row_heads * HD, kv_stride = (size_t)kv_row_heads * HD;
+    const size_t q_stride = q_row_elems, kv_stride = kv_row_elems;
     int k_first, n_tiles;
     key_tiles(q0, len, window, k_first, n_tiles, start);
     const int np = pf::parts_of(n_tiles, parts, piece);
@@ -292,6 +292,11 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q_src, const bf16* __restrict__
         }
         return;
     }
+    if (sinks != nullptr) {                           // a key of that score without a value
+        const float z = sinks[head] * LOG2E;
+        l_run[0] += ex2(z - m_run[0]);
+        l_run[1] += ex2(z - m_run[1]);
+    }
     const float inv_lo = 1.0f / l_run[0], inv_hi = 1.0f / l_run[1];
     bf16* out_lo = out + (size_t)(first + row_lo - start) * nq * HD + (size_t)head * HD + t * 2;
     bf16* out_hi = out + (size_t)(first + row_hi - start) * nq * HD + (size_t)head * HD + t * 2;
@@ -312,7 +317,7 @@ constexpr int MERGE_ROWS = 8;                         // rows of the tile per CT
 __global__ void __launch_bounds__(256)
 attn_prefill_merge_kernel(const float* __restrict__ partial, const int* __restrict__ seq_first_row,
                           const int* __restrict__ seq_len, int n_seq, bf16* __restrict__ out, int nq, int window,
-                          int parts, int piece, const int* __restrict__ seq_start) {
+                          int parts, int piece, const int* __restrict__ seq_start, const float* __restrict__ sinks) {
     const int gtile = blockIdx.x, head = blockIdx.y;
     const int r_begin = blockIdx.z * MERGE_ROWS;
     // the step's tables were written before the attention kernel started: they are read while it still runs
@@ -356,6 +361,7 @@ attn_prefill_merge_kernel(const float* __restrict__ partial, const int* __restri
             l += lp[p] * w;
             acc[0] += a[p].x * w; acc[1] += a[p].y * w; acc[2] += b[p].x * w; acc[3] += b[p].y * w;
         }
+        if (sinks != nullptr) l += ex2(sinks[head] * 1.4426950408889634f - m);
         const float inv = 1.0f / l;
         bf16* o = out + (size_t)(first + q0 + r) * nq * HD + (size_t)head * HD + c;
         *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16(acc[0] * inv, acc[1] * inv), pack_bf16(acc[2] * inv, acc[3] * inv));
@@ -499,13 +505,19 @@ JANIS_EXPORT void janis_attn_set_prefill_kernel(int which) { g_prefill_kernel = 
 // seq_len then holds the lengths after the step, seq_first_row the row of a sequence's first token of this step, and
 // keys and values of positions below seq_start come from the cache line (kpool, vpool, page_table, ring_len as in
 // janis_attn_decode); such a step runs on the mma.sync kernel.
+// q_row_elems, kv_row_elems: elements between neighbouring rows, where rows hold more than whole heads (0: the row heads
+// times the head size).  sinks ([nq] floats, or null): exp(sinks[h]) joins head h's denominator.
 JANIS_EXPORT int janis_attn_prefill_mma(const void* q_src, const void* kv_src, int n_tok, const int* seq_first_row,
                                         const int* seq_len, int n_seq, int n_tiles_bound, void* out, int nq,
                                         int nkv, int q_row_heads, int kv_row_heads, int kv_k_head0, float scale,
                                         float cap, int window, float* partial, long long partial_floats,
                                         const int* seq_start, const int* seq_slot, const void* kpool, const void* vpool,
                                         const int* page_table, int table_stride, int ring_len, int max_len,
-                                        cudaStream_t stream) {
+                                        int q_row_elems, int kv_row_elems, const float* sinks, cudaStream_t stream) {
+    if (q_row_elems == 0) q_row_elems = q_row_heads * pf::HD;
+    if (kv_row_elems == 0) kv_row_elems = kv_row_heads * pf::HD;
+    if (q_row_elems % 8 || kv_row_elems % 8 || q_row_elems < nq * pf::HD || kv_row_elems < (kv_k_head0 + 2 * nkv) * pf::HD)
+        return fail("attn_prefill_mma: rows of %d and %d elements do not hold the heads", q_row_elems, kv_row_elems);
     if (n_seq <= 0 || n_tiles_bound <= 0) return 0;
     if (nkv <= 0 || nq % nkv) return fail("attn_prefill_mma: %d query heads do not divide over %d key heads", nq, nkv);
     if (((uintptr_t)q_src | (uintptr_t)kv_src | (uintptr_t)out | (uintptr_t)partial | (uintptr_t)kpool | (uintptr_t)vpool) & 15)
@@ -549,20 +561,20 @@ JANIS_EXPORT int janis_attn_prefill_mma(const void* q_src, const void* kv_src, i
     int done = -1;
     if (g_prefill_kernel == 1 && !ext)                // the tcgen05 kernel takes sequences that start at position 0
         done = launch_prefill_tc05(q_src, kv_src, n_tok, seq_first_row, seq_len, n_seq, n_tiles_bound, out, nq, nkv,
-                                   q_row_heads, kv_row_heads, kv_k_head0, scale, cap, window, parts, piece, partial,
-                                   stream);
+                                   q_row_elems, kv_row_elems, kv_k_head0, scale, cap, window, parts, piece, partial,
+                                   sinks, stream);
     if (done > 0) return 1;
     if (done < 0) {
         dim3 grid(nq, n_tiles_bound * parts);
         auto kernel = ext ? pf::attn_prefill_mma_kernel<true> : pf::attn_prefill_mma_kernel<false>;
         if (launch_kernel("attn_prefill_mma", kernel, grid, dim3(pf::THREADS), pf::SMEM_BYTES, stream, 1, (const bf16*)q_src,
-                          (const bf16*)kv_src, seq_first_row, seq_len, n_seq, (bf16*)out, nq, nkv, q_row_heads,
-                          kv_row_heads, kv_k_head0, scale, cap, window, parts, piece, partial, cached))
+                          (const bf16*)kv_src, seq_first_row, seq_len, n_seq, (bf16*)out, nq, nkv, q_row_elems,
+                          kv_row_elems, kv_k_head0, scale, cap, window, parts, piece, partial, cached, sinks))
             return 1;
     }
     g_prefill_kernels = parts == 1 ? 1 : 2;
     if (parts == 1) return 0;
     return launch_kernel("attn_prefill_merge", pf::attn_prefill_merge_kernel, dim3(n_tiles_bound, nq, pf::BM / pf::MERGE_ROWS), dim3(256), 0, stream, 1,
                          (const float*)partial, seq_first_row, seq_len, n_seq, (bf16*)out, nq, window, parts, piece,
-                         seq_start);
+                         seq_start, sinks);
 }

@@ -217,7 +217,7 @@ __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                          const int* __restrict__ seq_first_row, const int* __restrict__ seq_len, int n_seq,
                          bf16* __restrict__ out, int nq, int nkv, int kv_k_head0, float scale, float cap, int window,
-                         int parts, int piece, float* __restrict__ partial) {
+                         int parts, int piece, float* __restrict__ partial, const float* __restrict__ sinks) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) unsigned long long bars[N_BARS];
     __shared__ uint32_t tmem_slot;
@@ -553,6 +553,7 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                             make_uint4(o[j], o[j + 1], o[j + 2], o[j + 3]);
                 }
             } else {
+                if (sinks != nullptr) l_row += pf::ex2(sinks[head] * LOG2E - m_ref);      // a key of that score without a value
                 const float inv = 1.0f / l_row;
 #pragma unroll 1
                 for (int c = OCOLS * h; c < OCOLS * (h + 1); c += 16) {
@@ -661,7 +662,8 @@ __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc05_items_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                                const int* __restrict__ seq_first_row, const int* __restrict__ seq_len, int n_seq,
                                bf16* __restrict__ out, int nq, int nkv, int kv_k_head0, float scale, float cap, int window,
-                               int parts, int piece, float* __restrict__ partial, int n_places, int sched_slot) {
+                               int parts, int piece, float* __restrict__ partial, int n_places, int sched_slot,
+                               const float* __restrict__ sinks) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) unsigned long long bars[N_BARS_ITEMS];
     int* sched = g_sched[sched_slot];
@@ -1046,6 +1048,7 @@ attn_prefill_tc05_items_kernel(const __grid_constant__ CUtensorMap map_q, const 
                                 make_uint4(o[j], o[j + 1], o[j + 2], o[j + 3]);
                     }
                 } else {
+                    if (sinks != nullptr) l_row += pf::ex2(sinks[me.head] * LOG2E - m_ref);
                     const float inv = 1.0f / l_row;
 #pragma unroll 1
                     for (int c = OCOLS * h; c < OCOLS * (h + 1); c += 16) {
@@ -1167,13 +1170,13 @@ static int tc05_sm_count() {
 }
 
 int launch_prefill_tc05(const void* q_src, const void* kv_src, int n_tok, const int* seq_first_row, const int* seq_len,
-                        int n_seq, int n_tiles_bound, void* out, int nq, int nkv, int q_row_heads, int kv_row_heads,
+                        int n_seq, int n_tiles_bound, void* out, int nq, int nkv, int q_row_elems, int kv_row_elems,
                         int kv_k_head0, float scale, float cap, int window, int parts, int piece, float* partial,
-                        cudaStream_t stream) {
+                        const float* sinks, cudaStream_t stream) {
     if (!pt::SUPPORTED) return -1;
     CUtensorMap mq, mkv;
-    if (!pt::make_map(&mq, q_src, n_tok, q_row_heads * pt::HD, pt::BM) ||
-        !pt::make_map(&mkv, kv_src, n_tok, kv_row_heads * pt::HD, pt::BN))
+    if (!pt::make_map(&mq, q_src, n_tok, q_row_elems, pt::BM) ||
+        !pt::make_map(&mkv, kv_src, n_tok, kv_row_elems, pt::BN))
         return -1;                                    // no encoder, or operands it refuses: the other kernel runs
     static bool configured = false;
     if (!configured) {
@@ -1208,12 +1211,12 @@ int launch_prefill_tc05(const void* q_src, const void* kv_src, int n_tok, const 
         auto items = cap > 0.f ? pt::attn_prefill_tc05_items_kernel<true> : pt::attn_prefill_tc05_items_kernel<false>;
         return launch_kernel("attn_prefill_tc05", items, dim3(ctas), dim3(pt::THREADS), pt::SMEM_BYTES, stream, 1, mq, mkv,
                              seq_first_row, seq_len, n_seq, (bf16*)out, nq, nkv, kv_k_head0, scale, cap, window, parts,
-                             piece, partial, n_places, slot);
+                             piece, partial, n_places, slot, sinks);
     }
     auto kernel = cap > 0.f ? pt::attn_prefill_tc05_kernel<true> : pt::attn_prefill_tc05_kernel<false>;
     return launch_kernel("attn_prefill_tc05", kernel, dim3(nq, n_tiles_bound * parts), dim3(pt::THREADS), pt::SMEM_BYTES,
                          stream, 1, mq, mkv, seq_first_row, seq_len, n_seq, (bf16*)out, nq, nkv, kv_k_head0, scale, cap,
-                         window, parts, piece, partial);
+                         window, parts, piece, partial, sinks);
 }
 
 int prefill_tc05_timeouts_async(int* host, cudaStream_t stream) {

@@ -73,8 +73,8 @@ __host__ __device__ __forceinline__ int parts_of(int n_tiles, int parts, int pie
 // The tcgen05 kernel of the same step (attention_prefill_tc05.cu): 0 launched, 1 failed (message set),
 // -1 this head size or these operands are not for it.
 int launch_prefill_tc05(const void* q_src, const void* kv_src, int n_tok, const int* seq_first_row, const int* seq_len,
-                        int n_seq, int n_tiles_bound, void* out, int nq, int nkv, int q_row_heads, int kv_row_heads,
+                        int n_seq, int n_tiles_bound, void* out, int nq, int nkv, int q_row_elems, int kv_row_elems,
                         int kv_k_head0, float scale, float cap, int window, int parts, int piece, float* partial,
-                        cudaStream_t stream);
+                        const float* sinks, cudaStream_t stream);
 
 }  // namespace janis

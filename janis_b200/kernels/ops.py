@@ -93,7 +93,8 @@ def attention_lib(head_dim: int):
         lib.janis_attn_prefill.argtypes = [P, P, I, P, P, P, P, I, I, I, I, I, I, F, F, I, P, P, P, P, P, I, I, P]
         lib.janis_attn_decode.argtypes = [P, P, P, I, P, I, P, P, P, c_longlong, P, I, I, I, I, F, F, I, I, I, I, P]
         lib.janis_attn_prefill_mma.argtypes = [P, P, I, P, P, I, I, P, I, I, I, I, I, F, F, I, P, c_longlong,
-                                               P, P, P, P, P, I, I, I, P]
+                                               P, P, P, P, P, I, I, I, I, I, P, P]
+        lib.janis_attn_decode_sinks.argtypes = [P, P, P, I, P, I, P, P, P, c_longlong, P, I, I, I, I, F, F, I, I, I, I, P, P]
         lib.janis_attn_set_prefill_kernel.argtypes = [I]
         lib.janis_attn_set_prefill_kernel.restype = None
         lib.janis_attn_set_prefill_piece.argtypes = [I]
@@ -687,9 +688,78 @@ def _attn_prefill_mma(qkv, seq_first_row, seq_len, out, nq, nkv, hd, scale, cap,
                                            qkv.shape[1], kv_row_heads, kv_k_head0, float(scale), float(cap),
                                            int(window), _t(scratch, "scratch", torch.float32) if scratch is not None else None,
                                            scratch.numel() if scratch is not None else 0, *cached,
-                                           max(int(n) for n in host_lens) if host_lens else 0, _stream()))
+                                           max(int(n) for n in host_lens) if host_lens else 0, 0, 0, None, _stream()))
     global _launches
     _launches += int(lib.janis_attn_prefill_kernels()) - 1     # the merge, when tiles were shared
+    return out
+
+
+def attn_rows_sizes(dtype, H: int, G: int, d: int, dv: int) -> bool:
+    """Whether `attn_prefill_rows` and `attn_decode_rows` take heads of these sizes."""
+    return dtype == torch.bfloat16 and d == dv and d % 16 == 0 and 16 <= d <= 256 and H % G == 0
+
+
+def attn_prefill_rows(rows, seq_first_row, seq_len, out, H: int, G: int, hd: int, scale: float, window: int = 0, cap: float = 0.0,
+                      sinks=None, scratch=None, host_lens=None, seq_start=None, seq_slot=None, kpool=None, vpool=None,
+                      page_table=None):
+    """`attn_prefill` (bfloat16, tensor cores) over rows that hold q (H heads), k and v (G heads each) first and anything
+    behind them; sinks [H] float32: exp of head h's number joins its denominator.  The line of a step that continues
+    sequences keeps every position (no ring); whether the step's own keys are stored already does not matter."""
+    T, width = rows.shape
+    _t(rows, "rows", torch.bfloat16, (T, None))
+    if width < (H + 2 * G) * hd or width % 8:
+        raise KernelError(f"attn_prefill_rows: rows of {width} elements for {H} + 2 x {G} heads of {hd}")
+    _t(out, "out", torch.bfloat16, (T, H * hd))
+    n_seq = seq_len.numel()
+    _t(seq_len, "seq_len", torch.int32, (n_seq,))
+    _t(seq_first_row, "seq_first_row", torch.int32, (n_seq,))
+    cached = _cached_args("attn_prefill_rows", seq_start, seq_slot, kpool, vpool, page_table, 0, torch.bfloat16, n_seq, G, hd)
+    lib = attention_lib(hd)
+    bm = lib.janis_attn_prefill_tile()
+    if host_lens is not None:
+        if len(host_lens) != n_seq or sum(host_lens) > T:
+            raise KernelError(f"attn_prefill_rows: host_lens {list(host_lens)} do not fit {n_seq} sequences of {T} tokens")
+        tiles = sum((int(n) + bm - 1) // bm for n in host_lens)
+    else:
+        tiles = (T + bm - 1) // bm + n_seq
+    need = int(lib.janis_attn_prefill_scratch(tiles, H))
+    if scratch is not None and (need == 0 or scratch.numel() < need):
+        scratch = None
+    _check(lib, lib.janis_attn_prefill_mma(rows.data_ptr(), rows.data_ptr(), T, seq_first_row.data_ptr(), seq_len.data_ptr(), n_seq,
+                                           tiles, out.data_ptr(), H, G, 0, 0, H, float(scale), float(cap), int(window),
+                                           _t(scratch, "scratch", torch.float32) if scratch is not None else None,
+                                           scratch.numel() if scratch is not None else 0, *cached,
+                                           max(int(n) for n in host_lens) if host_lens else 0, width, width,
+                                           _t(sinks, "sinks", torch.float32, (H,)) if sinks is not None else None, _stream()))
+    global _launches
+    _launches += int(lib.janis_attn_prefill_kernels()) - 1
+    return out
+
+
+def attn_decode_rows(rows, kpool, vpool, page_table, seq_slot, seq_len, scratch, out, H: int, G: int, hd: int, scale: float,
+                     window: int, chunk: int, max_chunks: int, cap: float = 0.0, sinks=None):
+    """`attn_decode` (bfloat16) for rows that hold the queries first and anything behind them, over a line that keeps every
+    position; sinks as in `attn_prefill_rows`."""
+    n_seq, width = rows.shape
+    _t(rows, "rows", torch.bfloat16, (n_seq, None))
+    if width < H * hd or width % 8:
+        raise KernelError(f"attn_decode_rows: rows of {width} elements for {H} heads of {hd}")
+    n_pages = kpool.shape[0]
+    _t(kpool, "kpool", torch.bfloat16, (n_pages, G, PAGE, hd))
+    _t(vpool, "vpool", torch.bfloat16, (n_pages, G, PAGE, hd))
+    _t(page_table, "page_table", torch.int32, (None, None))
+    _t(scratch, "scratch", torch.float32)
+    _t(out, "out", torch.bfloat16, (n_seq, H * hd))
+    if seq_slot.numel() < n_seq or seq_len.numel() < n_seq:
+        raise KernelError("attn_decode_rows: sequence tables shorter than the batch")
+    lib = attention_lib(hd)
+    direct = max_chunks == 1 and _decode_kernel.get(hd, 2) == 2
+    _check(lib, lib.janis_attn_decode_sinks(rows.data_ptr(), kpool.data_ptr(), vpool.data_ptr(), _DT[rows.dtype], page_table.data_ptr(),
+                                            page_table.shape[1], _t(seq_slot, "seq_slot", torch.int32),
+                                            _t(seq_len, "seq_len", torch.int32), scratch.data_ptr(), scratch.numel(), out.data_ptr(),
+                                            n_seq, H, G, width, float(scale), float(cap), int(window), 0, int(chunk), int(max_chunks),
+                                            _t(sinks, "sinks", torch.float32, (H,)) if sinks is not None else None, _stream()),
+           kernels=1 if direct else 2)
     return out
 
 

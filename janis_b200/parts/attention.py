@@ -27,6 +27,56 @@ from ..weights.loader import TensorSpec
 from .base import Mixer, PositionEncoding, Runtime, StepContext
 
 
+def decode_geometry(ctx: StepContext, sm_count: int, head_dim: int, n_kv_heads: int, window: int):
+    """(chunk, most chunks a sequence has): how the keys of a decode step are cut up for the CTAs.
+
+    A CTA per (sequence, key/value head, chunk); two or three CTAs fit an SM.  In tiles of 32 keys a CTA costs the tiles
+    of its chunk plus a fixed share for starting its pipeline and for the merge.  Long chunks amortise the fixed
+    share, short ones fill the SMs and even the load out.  The host knows the step's lengths by their bound,
+    their mean (in eighths of the bound) and whether they are about equal; all three are part of a recorded
+    step's key.  Measured on a B200 at 8 heads over 4, head size 256 (attention and merge, one layer): 64
+    sequences of 198 to 2,087 keys 63.6 us at chunks of 384 against 86.9 at 2,048 (one chunk a sequence); 8 such
+    sequences 14.4 us at 128 against 16.9 at 256; 8 sequences of 8,100 keys 49.5 us at 1,024."""
+    bound = max(ctx.len_bound, 1)
+    span = min(bound, window) if window else bound
+    pairs = ctx.n_seq * n_kv_heads
+    held = getattr(ctx.rt.ops, "attn_decode_resident", None)       # CTAs of a launch that the GPU holds at once
+    mean = min(ctx.len_mean or bound, bound)
+    seen = min(mean, window) if window else mean          # keys a sequence of mean length attends over
+    extra = 1 if window and seen >= window else 0         # a window seldom starts on a chunk's border
+    best = None
+    for chunk in range(64, 2049, 64):
+        launched = (bound + chunk - 1) // chunk
+        if window:
+            launched = min(launched, (window + chunk - 1) // chunk + 1)
+        resident = held(head_dim, ctx.rt.dtype, pairs * launched, sm_count) if held else 2 * sm_count
+        if ctx.len_even:
+            # CTAs of equal length run in waves.  A launch of no more CTAs than SMs takes stages of 64 keys at
+            # head sizes above 128, which cost about two thirds of two stages of 32 (one sequence of 8,100 keys:
+            # 14.9 us a layer at chunks of 256 and 128 CTAs against 17.1 at chunks of 192 and 172 CTAs)
+            n_chunks = (seen + chunk - 1) // chunk + extra
+            waves = (pairs * n_chunks + resident - 1) // resident
+            wide = head_dim > 128 and pairs * launched <= sm_count
+            cost = waves * (min(chunk, seen) // 32 * (0.65 if wide else 1.0) + 6) + n_chunks / 8      # (the merge reads every chunk)
+        else:
+            # unequal lengths: the SMs' even share of all tiles and fixed shares, then the longest CTA, which
+            # may start last (halved while every CTA has an SM's slot to itself from the start)
+            n_ctas = pairs * (seen / chunk + 0.5 + extra)
+            share = (4 * n_ctas + pairs * seen / 32) / resident
+            cost = min(chunk, span) // 32 + 4 + (share if n_ctas > resident else share / 2) + (span / chunk + extra) / 8
+        if chunk < bound:
+            cost += 6          # more than one chunk a sequence: partial results and a merge kernel
+        if (min(bound, span) + chunk - 1) // chunk + (1 if window and span >= window else 0) > 64:
+            cost += 8          # beyond 64 chunks the merge forms its weights block-wide, not per warp: twice the time
+        if best is None or cost < best[0]:
+            best = (cost, chunk)
+    chunk = best[1]
+    max_chunks = (bound + chunk - 1) // chunk
+    if window:
+        max_chunks = min(max_chunks, (window + chunk - 1) // chunk + 1)
+    return chunk, max_chunks
+
+
 class SoftmaxAttention(Mixer):
     def __init__(self, hidden: int, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                  position: PositionEncoding, names: dict[str, str], softcap: float = 0.0,
@@ -83,53 +133,7 @@ class SoftmaxAttention(Mixer):
 
     # -- a step ------------------------------------------------------------
     def _decode_geometry(self, ctx: StepContext, sm_count: int):
-        """(chunk, most chunks a sequence has): how the keys of a decode step are cut up for the CTAs.
-
-        A CTA per (sequence, key/value head, chunk); two or three CTAs fit an SM.  In tiles of 32 keys a CTA costs the tiles
-        of its chunk plus a fixed share for starting its pipeline and for the merge.  Long chunks amortise the fixed
-        share, short ones fill the SMs and even the load out.  The host knows the step's lengths by their bound,
-        their mean (in eighths of the bound) and whether they are about equal; all three are part of a recorded
-        step's key.  Measured on a B200 at 8 heads over 4, head size 256 (attention and merge, one layer): 64
-        sequences of 198 to 2,087 keys 63.6 us at chunks of 384 against 86.9 at 2,048 (one chunk a sequence); 8 such
-        sequences 14.4 us at 128 against 16.9 at 256; 8 sequences of 8,100 keys 49.5 us at 1,024."""
-        bound = max(ctx.len_bound, 1)
-        span = min(bound, self.window) if self.window else bound
-        pairs = ctx.n_seq * self.n_kv_heads
-        held = getattr(ctx.rt.ops, "attn_decode_resident", None)       # CTAs of a launch that the GPU holds at once
-        mean = min(ctx.len_mean or bound, bound)
-        seen = min(mean, self.window) if self.window else mean          # keys a sequence of mean length attends over
-        extra = 1 if self.window and seen >= self.window else 0         # a window seldom starts on a chunk's border
-        best = None
-        for chunk in range(64, 2049, 64):
-            launched = (bound + chunk - 1) // chunk
-            if self.window:
-                launched = min(launched, (self.window + chunk - 1) // chunk + 1)
-            resident = held(self.head_dim, ctx.rt.dtype, pairs * launched, sm_count) if held else 2 * sm_count
-            if ctx.len_even:
-                # CTAs of equal length run in waves.  A launch of no more CTAs than SMs takes stages of 64 keys at
-                # head sizes above 128, which cost about two thirds of two stages of 32 (one sequence of 8,100 keys:
-                # 14.9 us a layer at chunks of 256 and 128 CTAs against 17.1 at chunks of 192 and 172 CTAs)
-                n_chunks = (seen + chunk - 1) // chunk + extra
-                waves = (pairs * n_chunks + resident - 1) // resident
-                wide = self.head_dim > 128 and pairs * launched <= sm_count
-                cost = waves * (min(chunk, seen) // 32 * (0.65 if wide else 1.0) + 6) + n_chunks / 8      # (the merge reads every chunk)
-            else:
-                # unequal lengths: the SMs' even share of all tiles and fixed shares, then the longest CTA, which
-                # may start last (halved while every CTA has an SM's slot to itself from the start)
-                n_ctas = pairs * (seen / chunk + 0.5 + extra)
-                share = (4 * n_ctas + pairs * seen / 32) / resident
-                cost = min(chunk, span) // 32 + 4 + (share if n_ctas > resident else share / 2) + (span / chunk + extra) / 8
-            if chunk < bound:
-                cost += 6          # more than one chunk a sequence: partial results and a merge kernel
-            if (min(bound, span) + chunk - 1) // chunk + (1 if self.window and span >= self.window else 0) > 64:
-                cost += 8          # beyond 64 chunks the merge forms its weights block-wide, not per warp: twice the time
-            if best is None or cost < best[0]:
-                best = (cost, chunk)
-        chunk = best[1]
-        max_chunks = (bound + chunk - 1) // chunk
-        if self.window:
-            max_chunks = min(max_chunks, (self.window + chunk - 1) // chunk + 1)
-        return chunk, max_chunks
+        return decode_geometry(ctx, sm_count, self.head_dim, self.n_kv_heads, self.window)
 
     def forward(self, x, ctx: StepContext, line):
         rt, ws, ops = ctx.rt, ctx.ws, ctx.rt.ops

@@ -29,8 +29,11 @@ per head): exp(sink_h) joins the denominator instead of 1.  The position encodin
 (1 - m) v + m v_first with the stored number m (names["vmix"]) before they are cached, v_first being the values of the
 same token in the layer that left them.
 
+In the serving dtype an attention without head mixing, blocks, turned values or kept positions, with values as wide as
+its keys, runs the kernels of `SoftmaxAttention` (a prompt step reads its own keys and values from the projected rows).
+
 Keys and values live in a paged cache line with separate head sizes.  A step writes its keys and values first
-and then attends over the line alone, so a prompt, a prompt that continues, a decode step and a layer that reads
+and then (but for those kernels) attends over the line alone, so a prompt, a prompt that continues, a decode step and a layer that reads
 the line of another layer (`own_kv=False`: queries only, no key/value tensors of its own) are one code path.
 Scores, the mixing, the softmax and the sums are float32 whatever the activations are.
 """
@@ -41,6 +44,7 @@ import torch
 from ..cache.cache import KVNeed
 from ..weights.loader import TensorSpec
 from .base import Mixer, Runtime, StepContext
+from .attention import decode_geometry
 from .position import RotaryEncoding
 
 
@@ -220,6 +224,8 @@ class TalkingHeadsAttention(Mixer):
                                  inv_v, H, G, d, dv, kv.k if self.own_kv else None, kv.v if self.own_kv else None,
                                  kv.table if self.own_kv else None, store=self.own_kv, **extras)
         att = ws.buf("tattn.ctx", (T, H * dv), rt.dtype)
+        if self._plain_heads(rt):
+            return self._attend_plain(rows, ctx, kv, att)
         more = {}
         if self.keep_first:
             more["keep_first"] = self.keep_first
@@ -250,3 +256,23 @@ class TalkingHeadsAttention(Mixer):
         return ops.talk_attention(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, kv.k, kv.v, kv.table, self.talk, inv_v, att,
                                   H, G, d, dv, self.scale, self.block, self.sink, one_row=decode, max_keys=max_keys,
                                   n_chunks=n_chunks, scratch=scratch, window=self.window, **more)
+
+    def _plain_heads(self, rt) -> bool:
+        """Whether the kernels of whole heads (one head a CTA, keys and values of one size) take this attention."""
+        return (self.talk is None and not self.block and self.value_position is None and not self.keep_first and self.own_kv
+                and not self.values_from_keys and (not self.sink or self.sink_values is not None) and hasattr(rt.ops, "attn_rows_sizes")
+                and rt.ops.attn_rows_sizes(rt.dtype, self.n_heads, self.n_kv_heads, self.key_dim, self.value_dim))
+
+    def _attend_plain(self, rows, ctx: StepContext, kv, att):
+        rt, ws, ops = ctx.rt, ctx.ws, ctx.rt.ops
+        H, G, d = self.n_heads, self.n_kv_heads, self.key_dim
+        if ctx.mode == "decode":
+            chunk, max_chunks = decode_geometry(ctx, rt.sm_count, d, G, self.window)
+            scratch = ws.buf("attn.partial", (ops.attn_decode_scratch_floats(ctx.n_seq, H, d, max_chunks),), torch.float32)
+            return ops.attn_decode_rows(rows, kv.k, kv.v, kv.table, ctx.seq_slot, ctx.seq_end, scratch, att, H, G, d, self.scale,
+                                        self.window, chunk, max_chunks, sinks=self.sink_values)
+        n_scratch = ops.attn_prefill_scratch_floats(ctx.n_tok, ctx.n_seq, H, d, rt.dtype)
+        scratch = ws.buf("attn.prefill_partial", (n_scratch,), torch.float32) if n_scratch else None
+        before = dict(seq_start=ctx.seq_start, seq_slot=ctx.seq_slot, kpool=kv.k, vpool=kv.v, page_table=kv.table) if ctx.extends else {}
+        return ops.attn_prefill_rows(rows, ctx.seq_first_row, ctx.seq_end, att, H, G, d, self.scale, self.window,
+                                     sinks=self.sink_values, scratch=scratch, host_lens=ctx.step_lens, **before)

@@ -412,6 +412,11 @@ def talk_attention(q_rows, tok_pos, tok_seq, seq_slot, kpool, vpool, page_table,
     return out
 
 
+def attn_rows_sizes(dtype, H, G, d, dv):
+    """The kernels of whole heads over longer rows state nothing new (a prompt or decode step of `talk_attention`)."""
+    return False
+
+
 def talk_attention_scratch_floats(T, n_chunks, H, dv):
     return T * n_chunks * H * (dv + 2) if n_chunks > 1 else 0
 

@@ -471,6 +471,76 @@ def test_attention_with_learnt_sinks_against_its_statement(dtype, H, G, d, dv):
 
 
 @GPU
+@pytest.mark.parametrize("H,G,d,window", [(4, 2, 16, 0), (8, 8, 64, 50), (8, 4, 128, 0), (6, 2, 48, 130), (4, 2, 256, 0), (5, 1, 80, 0),
+                                          (16, 1, 192, 0)])
+def test_kernels_of_whole_heads_over_longer_rows_with_learnt_sinks(H, G, d, window):
+    """Prompt steps (every form of the kernels; sequences that start and sequences that go on from stored keys) and decode
+    steps (a row's keys in one chunk and in several), with columns behind q, k and v, with and without sinks."""
+    from janis_b200.kernels import ops
+    from tests import kernel_refs as R
+    dtype = torch.bfloat16
+    g = torch.Generator().manual_seed(13)
+    width = ((H + 2 * G) * d + 9 + 7) // 8 * 8
+    scale = 2.0 * d ** -0.5
+    sinks = torch.randn(H, generator=g)
+    sinks[0], sinks[1] = 6.0, -30.0
+
+    def case(lens, starts):
+        tok_pos, tok_seq, slots, first, start, end = _tables(lens, starts, [(3 * s + 1) % (len(lens) + 1) for s in range(len(lens))])
+        per = max(-(-(a + n) // ops.PAGE) for a, n in zip(starts, lens))
+        n_slots = len(lens) + 1
+        table = torch.randperm(n_slots * per, generator=g).view(n_slots, per).to(torch.int32)
+        kp = torch.randn(n_slots * per, G, ops.PAGE, d, generator=g).to(dtype)
+        vp = torch.randn(n_slots * per, G, ops.PAGE, d, generator=g).to(dtype)
+        rows = torch.randn(sum(lens), width, generator=g).to(dtype)
+        R.qkv_rotate_store(rows, tok_pos, tok_seq, slots, torch.zeros(0), 0, None, H, G, d, d, kp, vp, table)
+        return tok_pos, tok_seq, slots, first, start, end, table, kp, vp, rows
+
+    def statement(c, z):
+        tok_pos, tok_seq, slots, first, start, end, table, kp, vp, rows = c
+        want = torch.zeros(rows.shape[0], H * d, dtype=dtype)
+        R.talk_attention(rows, tok_pos, tok_seq, slots, kp, vp, table, None, None, want, H, G, d, d, scale, 0, z is not None,
+                         window=window, sink_values=z)
+        return want
+
+    for lens, starts in (([1, 70, 129, 300], [0] * 4), ([200, 2, 65], [70, 129, 0])):
+        c = case(lens, starts)
+        tok_pos, tok_seq, slots, first, start, end, table, kp, vp, rows = c
+        before = dict(seq_start=start.cuda(), seq_slot=slots.cuda(), kpool=kp.cuda(), vpool=vp.cuda(), page_table=table.cuda()) if any(starts) else {}
+        T = rows.shape[0]
+        n = ops.attn_prefill_scratch_floats(T, len(lens), H, d, dtype)
+        for z in (sinks, None):
+            want = statement(c, z)
+            for which in (0, 1, 2, 3):
+                for piece in (0, 1):
+                    ops.attn_set_prefill_kernel(d, which)
+                    ops.attn_set_prefill_piece(d, piece)
+                    try:
+                        got = torch.full((T, H * d), float("nan"), dtype=dtype, device="cuda")
+                        ops.attn_prefill_rows(rows.cuda(), first.cuda(), end.cuda(), got, H, G, d, scale, window,
+                                              sinks=z.cuda() if z is not None else None,
+                                              scratch=torch.full((max(n, 1),), float("nan"), device="cuda") if n else None,
+                                              host_lens=tuple(lens) if which != 2 else None, **before)
+                    finally:
+                        ops.attn_set_prefill_kernel(d, 1)
+                        ops.attn_set_prefill_piece(d, 0)
+                    _close(got, want, dtype, ("prompt", lens, which, piece, z is not None))
+        assert ops.attn_tc05_timeouts(d) == 0
+    c = case([1] * 5, [0, 63, 64, 200, 299])
+    tok_pos, tok_seq, slots, first, start, end, table, kp, vp, rows = c
+    for z in (sinks, None):
+        want = statement(c, z)
+        for chunk in (64, 128, 320):
+            chunks = -(-320 // chunk)
+            scratch = torch.full((ops.attn_decode_scratch_floats(5, H, d, chunks),), float("nan"), device="cuda")
+            got = torch.full((5, H * d), float("nan"), dtype=dtype, device="cuda")
+            ops.attn_decode_rows(*_cuda(rows, kp, vp, table, slots, end), scratch, got, H, G, d, scale, window, chunk, chunks,
+                                 sinks=z.cuda() if z is not None else None)
+            _close(got, want, dtype, ("decode", chunk, z is not None))
+    assert ops.attn_wait_timeouts(d) == 0
+
+
+@GPU
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("C,K,off", [(48, 4, 48), (21, 5, 3), (256, 2, 0), (10, 1, 4), (600, 4, 8)])
 def test_filter_with_a_bias_on_its_inputs_against_its_statement(dtype, C, K, off):

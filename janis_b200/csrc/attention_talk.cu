@@ -142,6 +142,107 @@ qkv_rotate_store_kernel(T* __restrict__ rows, int row_elems, const int* __restri
         }
 }
 
+// The same, 16 bytes of a row at a time (every head's turned part, its rest and the values are whole 16-byte pieces at
+// 16-byte borders; values are not turned): a thread an item, which is a run of pairs (two pieces), a piece of what does not
+// turn, or a piece of the values.  A decode step's few CTAs then have one or two items a thread instead of a head a warp.
+template <typename T>
+__global__ void __launch_bounds__(256)
+qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __restrict__ tok_pos,
+                            const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
+                            const float* __restrict__ inv_qk, int rot, int H, int G, int d, int dv, int with_kv,
+                            T* __restrict__ kpool, T* __restrict__ vpool, const int* __restrict__ page_table,
+                            int table_stride, RotateExtras ex, T* __restrict__ v_first) {
+    constexpr int V = Vec16<T>::N;
+    extern __shared__ float2 turn_s[];
+    const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+    const int hq = rot >> 1, n_heads = with_kv ? H + G : H;
+    grid_dependents_launch();
+    const int pos = tok_pos[t];
+    T* kdst = nullptr;
+    T* vdst = nullptr;
+    if (with_kv) {
+        const int slot = seq_slot[tok_seq[t]];
+        if (slot >= 0) {
+            const int page = page_table[(size_t)slot * table_stride + pos / JANIS_PAGE];
+            kdst = kpool + ((size_t)page * G * JANIS_PAGE + pos % JANIS_PAGE) * d;
+            vdst = vpool + ((size_t)page * G * JANIS_PAGE + pos % JANIS_PAGE) * dv;
+        }
+    }
+    for (int i = tid; i < hq; i += nt) {
+        float s, c;
+        sincosf((float)pos * inv_qk[i], &s, &c);
+        turn_s[i] = make_float2(s * ex.amp, c * ex.amp);
+    }
+    __syncthreads();
+    grid_dependency_wait();
+    T* row = rows + (size_t)t * row_elems;
+    auto add_bias = [&](float (&x)[V], int at) {
+        if (ex.bias == nullptr) return;
+#pragma unroll
+        for (int e = 0; e < V; e += 4) {
+            float b[4];
+            Vec16<float>::load(ex.bias + at + e, b);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) x[e + q] += b[q];
+        }
+    };
+    const int per_turn = hq / V, per_rest = (d - rot) / V, per_v = dv / V;
+    const int n_turn = n_heads * per_turn;
+    const int rest0 = ex.bias != nullptr ? 0 : H;                    // (without a bias the queries' rest stays as it is)
+    const int n_rest = n_heads > rest0 ? (n_heads - rest0) * per_rest : 0, n_val = with_kv ? G * per_v : 0;
+    for (int u = tid; u < n_turn + n_rest + n_val; u += nt) {
+        if (u < n_turn) {
+            const int head = u / per_turn, i = (u - head * per_turn) * V, at = head * d + i;
+            float a[V], b[V];
+            Vec16<T>::load(row + at, a);
+            Vec16<T>::load(row + at + hq, b);
+            add_bias(a, at);
+            add_bias(b, at + hq);
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                const float2 sc = turn_s[i + e];
+                float lo, hi;
+                rotate_pair(a[e], b[e], sc.x, sc.y, lo, hi);
+                a[e] = lo;
+                b[e] = hi;
+            }
+            Vec16<T>::store(row + at, a);
+            Vec16<T>::store(row + at + hq, b);
+            if (head >= H && kdst != nullptr) {
+                T* kd = kdst + (size_t)(head - H) * JANIS_PAGE * d + i;
+                Vec16<T>::store(kd, a);
+                Vec16<T>::store(kd + hq, b);
+            }
+        } else if (u < n_turn + n_rest) {
+            const int w = u - n_turn, head = rest0 + w / per_rest, c = rot + (w % per_rest) * V, at = head * d + c;
+            float a[V];
+            Vec16<T>::load(row + at, a);
+            if (ex.bias != nullptr) {
+                add_bias(a, at);
+                Vec16<T>::store(row + at, a);
+            }
+            if (head >= H && kdst != nullptr) Vec16<T>::store(kdst + (size_t)(head - H) * JANIS_PAGE * d + c, a);
+        } else {
+            const int w = u - n_turn - n_rest, g = w / per_v, c = (w - g * per_v) * V, at = (H + G) * d + g * dv + c;
+            float a[V];
+            Vec16<T>::load(row + at, a);
+            if (ex.bias != nullptr || ex.mix != 0) {
+                add_bias(a, at);
+                T* first = v_first + ((size_t)t * G + g) * dv + c;
+                if (ex.mix == 2) {
+                    float f[V];
+                    Vec16<T>::load(first, f);
+#pragma unroll
+                    for (int e = 0; e < V; ++e) a[e] = fmaf(ex.share, f[e], (1.f - ex.share) * a[e]);
+                }
+                Vec16<T>::store(row + at, a);
+                if (ex.mix == 1) Vec16<T>::store(first, a);
+            }
+            if (vdst != nullptr) Vec16<T>::store(vdst + (size_t)g * JANIS_PAGE * dv + c, a);
+        }
+    }
+}
+
 // ---------------------------------------------------------------------------
 // The plain kernel: one CTA per query token, all heads together, tiles of up to 32 keys staged in shared
 // memory as floats.  It is the 32-bit path, and the bfloat16 path of sizes the tensor-core kernel leaves out.
@@ -846,6 +947,20 @@ JANIS_EXPORT int janis_qkv_rotate_store(void* rows, int dtype, int row_elems, co
     const size_t bytes = ((size_t)(rot >> 1) + (inv_v != nullptr ? dv >> 1 : 0)) * sizeof(float2);
     if (bytes > 48 * 1024) return fail("qkv_rotate_store: %zu bytes of angles", bytes);
     const RotateExtras ex = {bias, amp, mix, share};
+    const int vec = dtype == JANIS_F32 ? 4 : 8;
+    if (inv_v == nullptr && (rot >> 1) % vec == 0 && d % vec == 0 && dv % vec == 0 && row_elems % vec == 0 &&
+        (((uintptr_t)rows | (uintptr_t)kpool | (uintptr_t)vpool | (uintptr_t)bias | (uintptr_t)v_first) & 15) == 0) {
+        const int items = ((with_kv ? H + G : H) * (d - rot / 2) + (with_kv ? G * dv : 0)) / vec;
+        const dim3 vgrid(T), vblock(items > 128 || T <= 64 ? 256 : 128);
+        if (dtype == JANIS_F32)
+            return launch_kernel("qkv_rotate_store", qkv_rotate_store_vec_kernel<float>, vgrid, vblock, bytes, stream, 1, (float*)rows,
+                                 row_elems, tok_pos, tok_seq, seq_slot, inv_qk, rot, H, G, d, dv, with_kv, (float*)kpool,
+                                 (float*)vpool, page_table, table_stride, ex, (float*)v_first);
+        if (dtype == JANIS_BF16)
+            return launch_kernel("qkv_rotate_store", qkv_rotate_store_vec_kernel<bf16>, vgrid, vblock, bytes, stream, 1, (bf16*)rows,
+                                 row_elems, tok_pos, tok_seq, seq_slot, inv_qk, rot, H, G, d, dv, with_kv, (bf16*)kpool,
+                                 (bf16*)vpool, page_table, table_stride, ex, (bf16*)v_first);
+    }
     const dim3 grid(T), block(128);
     if (dtype == JANIS_F32)
         return launch_kernel("qkv_rotate_store", qkv_rotate_store_kernel<float>, grid, block, bytes, stream, 1, (float*)rows,

@@ -14,8 +14,6 @@
 
 namespace janis {
 
-constexpr int REC_THREADS = 256;
-
 __device__ __forceinline__ float logistic(float v) { return 1.0f / (1.0f + expf(-v)); }
 
 // one token's decay minus one and input
@@ -32,19 +30,19 @@ struct RecurrenceShape {
     float scale;
 };
 
-// A CTA per (CH channels, sequence).  Its 256 / CH groups of threads take runs of TT tokens: each runs its tokens from a
+// A CTA per (CH channels, sequence).  Its NT / CH groups of threads take runs of TT tokens: each runs its tokens from a
 // state of zero, keeping every token's state and the product of the decays so far (minus one); the groups' totals meet in
 // shared memory (two buffers that take turns, one barrier a round), every thread carries the state over all groups in
 // order and puts the state that enters its own group under its tokens.  The inputs of the next round are on their way
 // while this one is computed.
-template <typename T, int CH, int TT>
-__global__ void __launch_bounds__(REC_THREADS)
+template <typename T, int CH, int TT, int NT>
+__global__ void __launch_bounds__(NT)
 gated_recurrence_scan_kernel(const T* __restrict__ u, const float* __restrict__ gates, const float* __restrict__ br,
                              const float* __restrict__ bi, const float* __restrict__ decay, const T* __restrict__ y_rows,
                              const float* __restrict__ yb, RecurrenceShape g, const int* __restrict__ seq_slot,
                              const int* __restrict__ seq_first_row, const int* __restrict__ seq_start,
                              const int* __restrict__ seq_end, float* __restrict__ state, T* __restrict__ out) {
-    constexpr int NG = REC_THREADS / CH, ROUND = NG * TT;
+    constexpr int NG = NT / CH, ROUND = NG * TT;
     __shared__ float2 tot_s[2][NG][CH];
     const int tid = threadIdx.x, cl = tid % CH, grp = tid / CH, seq = blockIdx.y;
     const int c_raw = blockIdx.x * CH + cl;
@@ -91,7 +89,7 @@ gated_recurrence_scan_kernel(const T* __restrict__ u, const float* __restrict__ 
         tot_s[buf][grp][cl] = make_float2(A, B);
         __syncthreads();
         float enter = S;
-#pragma unroll 4
+#pragma unroll 8
         for (int q = 0; q < NG; ++q) {
             if (q == grp) enter = S;
             const float2 ab = tot_s[buf][q][cl];
@@ -108,11 +106,27 @@ gated_recurrence_scan_kernel(const T* __restrict__ u, const float* __restrict__ 
     if (st != nullptr && live && grp == 0) *st = S;
 }
 
-// Steps of single rows (every sequence brings one token).  A CTA per (block of channels, 8 channels of it, 8 rows): the
-// rows' u of the block in shared memory as floats, a warp per channel, whose two rows of the gates' matrices it reads once,
-// 16 bytes a lane (the first piece before the kernel waits for its predecessor: weights are constants); the sums of the 8
-// rows meet in butterflies and lane r finishes row r.
-constexpr int REC_ROWS = 8, REC_WARPS = 8;
+// Steps of single rows (every sequence brings one token).  A CTA per (block of channels, 16 channels of it, 8 rows): the
+// rows' u of the block in shared memory as floats; 8 lanes share a channel, take its two rows of the gates' matrices 16
+// bytes at a time in turn (the first pieces before the kernel waits for its predecessor: weights are constants) and scatter
+// their partial sums so that lane r of the eight ends up with row r's, which it finishes.
+constexpr int REC_ROWS = 8, REC_WARPS = 4, REC_CHANNELS = REC_WARPS * 4;
+
+// v[0..7] of each of 8 lanes: the lanes' sums of v[own lane], in a fixed order
+__device__ __forceinline__ float scatter_sum8(float (&v)[REC_ROWS], int sub) {
+#pragma unroll
+    for (int half = 4; half >= 1; half >>= 1) {
+        const bool up = (sub & half) != 0;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            if (i < half) {
+                const float mine = up ? v[i + half] : v[i], other = up ? v[i] : v[i + half];
+                v[i] = mine + __shfl_xor_sync(0xffffffffu, other, half);
+            }
+        }
+    }
+    return v[0];
+}
 
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(REC_WARPS * 32)
@@ -120,80 +134,103 @@ gated_recurrence_rows_kernel(const T* __restrict__ u, const T* __restrict__ w, c
                              const float* __restrict__ bi, const float* __restrict__ decay, const T* __restrict__ y_rows,
                              const float* __restrict__ yb, RecurrenceShape g, const int* __restrict__ tok_seq,
                              const int* __restrict__ seq_slot, int n_rows, float* __restrict__ state, T* __restrict__ out) {
-    constexpr int V = Vec16<T>::N;
+    constexpr int V = Vec16<T>::N, AHEAD = 4;             // pieces asked for together
     extern __shared__ __align__(16) float rec_u[];        // [REC_ROWS][block]
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n = g.block;
-    const int b = blockIdx.x, j = blockIdx.y * REC_WARPS + warp, row0 = blockIdx.z * REC_ROWS, here = min(REC_ROWS, n_rows - row0);
-    const bool mine = j < n;
-    const int c = b * n + (mine ? j : 0);
-    const T* wr = w + ((size_t)b * 2 * n + (mine ? j : 0)) * n;
+    const int tid = threadIdx.x, lane = tid & 31, sub = lane & 7, n = g.block;
+    const int b = blockIdx.x, j_raw = blockIdx.y * REC_CHANNELS + (tid >> 3), row0 = blockIdx.z * REC_ROWS;
+    const int here = min(REC_ROWS, n_rows - row0);
+    const bool mine = j_raw < n;
+    const int j = mine ? j_raw : n - 1, c = b * n + j;    // (lanes without a channel repeat the last one and store nothing)
+    const T* wr = w + ((size_t)b * 2 * n + j) * n;
     const T* wi = wr + (size_t)n * n;
+    const bool live = mine && sub < here;
+    const int row = row0 + (sub < here ? sub : 0);
     grid_dependents_launch();
-    float fr[V], fi[V];
-    if (VEC && lane * V < n) {
-        Vec16<T>::load(wr + lane * V, fr);
-        Vec16<T>::load(wi + lane * V, fi);
+    uint4 pr[AHEAD], pi[AHEAD];
+    if (VEC) {
+#pragma unroll
+        for (int a = 0; a < AHEAD; ++a) {
+            const int k = (sub + 8 * a) * V;
+            if (k < n) {
+                pr[a] = *reinterpret_cast<const uint4*>(wr + k);
+                pi[a] = *reinterpret_cast<const uint4*>(wi + k);
+            }
+        }
     }
     const float brc = br[c], bic = bi[c], dec = decay[c], ybc = yb != nullptr ? yb[c] : 0.f;
-    const int slot = lane < here ? seq_slot[tok_seq[row0 + lane]] : -1;
+    const int slot = live ? seq_slot[tok_seq[row]] : -1;
     grid_dependency_wait();
-    float S = 0.f, y = 0.f, uc = 0.f;
-    if (mine && lane < here) {
-        if (slot >= 0) S = state[(size_t)slot * g.C + c];
-        y = to_float(y_rows[(size_t)(row0 + lane) * g.y_stride + g.y_off + c]);
-        uc = to_float(u[(size_t)(row0 + lane) * g.C + c]);
-    }
-    for (int k = tid; k < REC_ROWS * n; k += REC_WARPS * 32) {
-        const int r = k / n;
-        rec_u[k] = r < here ? to_float(u[(size_t)(row0 + r) * g.C + (size_t)b * n + k % n]) : 0.f;
+    const float S0 = slot >= 0 ? state[(size_t)slot * g.C + c] : 0.f;
+    const float y = to_float(y_rows[(size_t)row * g.y_stride + g.y_off + c]);
+    if (VEC) {
+        const int per = n / V;
+        for (int k = tid; k < REC_ROWS * per; k += REC_WARPS * 32) {
+            const int r = k / per, at = (k - r * per) * V;
+            float x[V];
+            if (r < here) Vec16<T>::load(u + (size_t)(row0 + r) * g.C + (size_t)b * n + at, x);
+#pragma unroll
+            for (int e = 0; e < V; e += 4) {
+                if (r >= here) x[e] = x[e + 1] = x[e + 2] = x[e + 3] = 0.f;
+                Vec16<float>::store(rec_u + r * n + at + e, x + e);
+            }
+        }
+    } else {
+        for (int k = tid; k < REC_ROWS * n; k += REC_WARPS * 32) {
+            const int r = k / n;
+            rec_u[k] = r < here ? to_float(u[(size_t)(row0 + r) * g.C + (size_t)b * n + k % n]) : 0.f;
+        }
     }
     __syncthreads();
-    if (!mine) return;
     float ar[REC_ROWS], ai[REC_ROWS];
 #pragma unroll
     for (int r = 0; r < REC_ROWS; ++r) ar[r] = ai[r] = 0.f;
     if (VEC) {
-        for (int k = lane * V; k < n; k += 32 * V) {
-            if (k != lane * V) {
-                Vec16<T>::load(wr + k, fr);
-                Vec16<T>::load(wi + k, fi);
-            }
+        for (int k0 = 0; k0 < n; k0 += 8 * V * AHEAD) {
 #pragma unroll
-            for (int r = 0; r < REC_ROWS; ++r) {
+            for (int a = 0; a < AHEAD; ++a) {
+                const int k = k0 + (sub + 8 * a) * V;
+                if (k < n) {
+                    float fr[V], fi[V];
+                    Vec16<T>::load(reinterpret_cast<const T*>(&pr[a]), fr);
+                    Vec16<T>::load(reinterpret_cast<const T*>(&pi[a]), fi);
 #pragma unroll
-                for (int e = 0; e < V; e += 4) {
-                    float x[4];
-                    Vec16<float>::load(rec_u + r * n + k + e, x);
+                    for (int r = 0; r < REC_ROWS; ++r) {
 #pragma unroll
-                    for (int q = 0; q < 4; ++q) {
-                        ar[r] = fmaf(fr[e + q], x[q], ar[r]);
-                        ai[r] = fmaf(fi[e + q], x[q], ai[r]);
+                        for (int e = 0; e < V; e += 4) {
+                            float x[4];
+                            Vec16<float>::load(rec_u + r * n + k + e, x);
+#pragma unroll
+                            for (int q = 0; q < 4; ++q) {
+                                ar[r] = fmaf(fr[e + q], x[q], ar[r]);
+                                ai[r] = fmaf(fi[e + q], x[q], ai[r]);
+                            }
+                        }
                     }
+                }
+                const int kn = k + 8 * V * AHEAD;             // the piece of the next round takes this one's place
+                if (kn < n) {
+                    pr[a] = *reinterpret_cast<const uint4*>(wr + kn);
+                    pi[a] = *reinterpret_cast<const uint4*>(wi + kn);
                 }
             }
         }
     } else {
-        for (int k = lane; k < n; k += 32) {
-            const float a = to_float(wr[k]), d = to_float(wi[k]);
+        for (int k = sub; k < n; k += 8) {
+            const float x0 = to_float(wr[k]), x1 = to_float(wi[k]);
 #pragma unroll
             for (int r = 0; r < REC_ROWS; ++r) {
-                ar[r] = fmaf(a, rec_u[r * n + k], ar[r]);
-                ai[r] = fmaf(d, rec_u[r * n + k], ai[r]);
+                ar[r] = fmaf(x0, rec_u[r * n + k], ar[r]);
+                ai[r] = fmaf(x1, rec_u[r * n + k], ai[r]);
             }
         }
     }
-    float zr = 0.f, zi = 0.f;
-#pragma unroll
-    for (int r = 0; r < REC_ROWS; ++r) {
-        const float a = warp_sum(ar[r]), d = warp_sum(ai[r]);
-        if (lane == r) zr = a, zi = d;
-    }
-    if (lane >= here) return;
+    const float zr = scatter_sum8(ar, sub), zi = scatter_sum8(ai, sub);
+    if (!live) return;
     float am1, in;
-    recurrence_terms(zr + brc, zi + bic, uc, dec, am1, in);
-    S = S + fmaf(S, am1, in);
+    recurrence_terms(zr + brc, zi + bic, to_float(u[(size_t)row * g.C + c]), dec, am1, in);
+    const float S = S0 + fmaf(S0, am1, in);
     if (slot >= 0) state[(size_t)slot * g.C + c] = S;
-    out[(size_t)(row0 + lane) * g.o_stride + g.o_off + c] = from_float<T>(g.scale * S * gelu_tanh(y + ybc));
+    out[(size_t)row * g.o_stride + g.o_off + c] = from_float<T>(g.scale * S * gelu_tanh(y + ybc));
 }
 
 }  // namespace janis
@@ -219,17 +256,17 @@ JANIS_EXPORT int janis_gated_recurrence_scan(const void* u, int dtype, const flo
     const RecurrenceShape g = {C, block, g_tok, g_block, y_stride, y_off, o_stride, o_off, scale};
     // narrow CTAs while wide ones would leave SMs idle
     const bool narrow = (long long)n_seq * ((C + 31) / 32) < 2 * 148;
-#define JANIS_REC(T, CH, TT)                                                                                           \
-    return launch_kernel("gated_recurrence_scan", gated_recurrence_scan_kernel<T, CH, TT>, dim3((C + CH - 1) / CH, n_seq), \
-                         dim3(REC_THREADS), 0, stream, 1, (const T*)u, gates, br, bi, decay, (const T*)y_rows, yb, g,  \
+#define JANIS_REC(T, CH, TT, NT)                                                                                       \
+    return launch_kernel("gated_recurrence_scan", gated_recurrence_scan_kernel<T, CH, TT, NT>, dim3((C + CH - 1) / CH, n_seq), \
+                         dim3(NT), 0, stream, 1, (const T*)u, gates, br, bi, decay, (const T*)y_rows, yb, g,  \
                          seq_slot, seq_first_row, seq_start, seq_end, state, (T*)out);
     if (dtype == JANIS_F32) {
-        if (narrow) JANIS_REC(float, 16, 4)
-        JANIS_REC(float, 32, 4)
+        if (narrow) JANIS_REC(float, 16, 4, 512)
+        JANIS_REC(float, 32, 4, 256)
     }
     if (dtype == JANIS_BF16) {
-        if (narrow) JANIS_REC(bf16, 16, 4)
-        JANIS_REC(bf16, 32, 4)
+        if (narrow) JANIS_REC(bf16, 16, 4, 512)
+        JANIS_REC(bf16, 32, 4, 256)
     }
 #undef JANIS_REC
     return fail("gated_recurrence_scan: unknown dtype %d", dtype);
@@ -243,7 +280,7 @@ JANIS_EXPORT int janis_gated_recurrence_rows(const void* u, int dtype, const voi
     if (recurrence_check("gated_recurrence_rows", C, block, y_stride, y_off, o_stride, o_off)) return 1;
     const size_t bytes = (size_t)REC_ROWS * block * sizeof(float);
     if (bytes > 48 * 1024) return fail("gated_recurrence_rows: blocks of %d channels do not fit shared memory", block);
-    const int blocks = C / block, gy = (block + REC_WARPS - 1) / REC_WARPS, gz = (n_rows + REC_ROWS - 1) / REC_ROWS;
+    const int blocks = C / block, gy = (block + REC_CHANNELS - 1) / REC_CHANNELS, gz = (n_rows + REC_ROWS - 1) / REC_ROWS;
     if (gy > 65535 || gz > 65535) return fail("gated_recurrence_rows: %d rows, blocks of %d", n_rows, block);
     const RecurrenceShape g = {C, block, 0, 0, y_stride, y_off, o_stride, o_off, scale};
     const int v = dtype == JANIS_F32 ? 4 : 8;

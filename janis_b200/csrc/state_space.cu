@@ -78,6 +78,95 @@ causal_conv_silu_kernel(const T* __restrict__ rows, int row_elems, int col_off, 
     }
 }
 
+// The same with 16 bytes of channels a thread, up to four taps: a thread takes its channels over a run of tokens in turn and
+// keeps the last K - 1 inputs in registers while the tokens are one sequence's; four tokens' inputs are asked for together.
+template <typename T>
+__global__ void __launch_bounds__(128)
+causal_conv_vec_kernel(const T* __restrict__ rows, int row_elems, int col_off, int C, int K,
+                       const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
+                       const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
+                       const int* __restrict__ seq_first_row, const int* __restrict__ seq_start,
+                       const int* __restrict__ seq_end, T* __restrict__ out, int n_tok, int run, int act,
+                       const float* __restrict__ in_bias) {
+    constexpr int V = Vec16<T>::N, KM = 4, AHEAD = 4;
+    const int per_row = C / V, idx = blockIdx.x * blockDim.x + threadIdx.x;
+    const int piece = idx / per_row, c = (idx - piece * per_row) * V, t0 = piece * run, t1 = min(n_tok, t0 + run);
+    grid_dependents_launch();
+    if (t0 >= n_tok) return;
+    float wk[KM][V], b[V], xb[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+        b[e] = bias != nullptr ? bias[c + e] : 0.f;
+        xb[e] = in_bias != nullptr ? in_bias[c + e] : 0.f;
+        if (K == KM) {
+            float row[KM];
+            Vec16<float>::load(w + (size_t)(c + e) * KM, row);
+#pragma unroll
+            for (int j = 0; j < KM; ++j) wk[j][e] = row[KM - 1 - j];
+        } else {
+#pragma unroll
+            for (int j = 0; j < KM; ++j) wk[j][e] = j < K ? w[(size_t)(c + e) * K + K - 1 - j] : 0.f;
+        }
+    }
+    grid_dependency_wait();
+    float past[KM - 1][V];                                   // past[j]: the input j + 1 tokens back
+    float* st = nullptr;
+    int seq = -1;
+    bool alone = false;
+    for (int tb = t0; tb < t1; tb += AHEAD) {
+        float x[AHEAD][V];
+#pragma unroll
+        for (int a = 0; a < AHEAD; ++a)
+            if (tb + a < t1) Vec16<T>::load(rows + (size_t)(tb + a) * row_elems + col_off + c, x[a]);
+#pragma unroll
+        for (int a = 0; a < AHEAD; ++a) {
+            const int t = tb + a;
+            if (t >= t1) break;
+            const int s = tok_seq[t];
+            if (s != seq) {                                  // the run enters a sequence: what lies before it
+                seq = s;
+                const int slot = seq_slot[s], i = t - seq_first_row[s];
+                alone = seq_end[s] - seq_start[s] == 1;
+                st = slot >= 0 ? state + (size_t)slot * max(K - 1, 1) * C + c : nullptr;
+#pragma unroll
+                for (int j = 0; j < KM - 1; ++j) {
+                    const int at = i - 1 - j;
+                    if (j < K - 1 && at >= 0) {
+                        Vec16<T>::load(rows + (size_t)(t - 1 - j) * row_elems + col_off + c, past[j]);
+#pragma unroll
+                        for (int e = 0; e < V; ++e) past[j][e] += xb[e];
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < V; ++e) past[j][e] = j < K - 1 && st != nullptr ? st[(size_t)(K - 1 + at) * C + e] : 0.f;
+                    }
+                }
+            }
+            float y[V];
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                x[a][e] += xb[e];
+                y[e] = fmaf(wk[0][e], x[a][e], b[e]);
+#pragma unroll
+                for (int j = 0; j < KM - 1; ++j)
+                    if (j < K - 1) y[e] = fmaf(wk[j + 1][e], past[j][e], y[e]);
+                if (act) y[e] = silu_f(y[e]);
+#pragma unroll
+                for (int j = KM - 2; j > 0; --j) past[j][e] = past[j - 1][e];
+                past[0][e] = x[a][e];
+            }
+            Vec16<T>::store(out + (size_t)t * C + c, y);
+            if (alone && st != nullptr) {                    // the sequence's only token of the step: the kept inputs move on
+#pragma unroll
+                for (int j = 0; j < KM - 1; ++j)
+                    if (j < K - 1) {
+#pragma unroll
+                        for (int e = 0; e < V; e += 4) Vec16<float>::store(st + (size_t)(K - 2 - j) * C + e, past[j] + e);
+                    }
+            }
+        }
+    }
+}
+
 // the K-1 inputs a sequence ends the step with: a thread per (sequence, channel) reads them all, then writes
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -463,7 +552,19 @@ static int conv_launch(const void* rows, int row_elems, int col_off, int C, int 
                        int act, const float* in_bias, cudaStream_t stream) {
     const int by = (C + 255) / 256, tpc = n_tok >= 1024 ? 8 : 1;
     if (by > 65535) return fail("causal_conv_silu: too many channels (%d)", C);
-    if (launch_kernel("causal_conv_silu", causal_conv_silu_kernel<T>, dim3((n_tok + tpc - 1) / tpc, by), dim3(256), 0, stream, 1,
+    constexpr int V = Vec16<T>::N;
+    if (K <= 4 && n_tok > 64 && C % V == 0 && col_off % V == 0 && row_elems % V == 0 &&
+        (((uintptr_t)rows | (uintptr_t)out | (uintptr_t)state | (uintptr_t)w) & 15) == 0) {
+        // (few rows: a thread a channel and token has less to do.)  Runs of tokens as long as every SM still gets two CTAs
+        const int per_row = C / V;
+        int run = 1;
+        while (run < 16 && (long long)((n_tok + 2 * run - 1) / (2 * run)) * per_row >= 148LL * 2 * 128) run *= 2;
+        const long long threads = (long long)((n_tok + run - 1) / run) * per_row;
+        if (launch_kernel("causal_conv_silu", causal_conv_vec_kernel<T>, dim3((unsigned)((threads + 127) / 128)), dim3(128), 0, stream, 1,
+                          (const T*)rows, row_elems, col_off, C, K, w, bias, state, tok_seq, seq_slot, seq_first_row, seq_start,
+                          seq_end, (T*)out, n_tok, run, act, in_bias))
+            return 1;
+    } else if (launch_kernel("causal_conv_silu", causal_conv_silu_kernel<T>, dim3((n_tok + tpc - 1) / tpc, by), dim3(256), 0, stream, 1,
                       (const T*)rows, row_elems, col_off, C, K, w, bias, state, tok_seq, seq_slot, seq_first_row, seq_start,
                       seq_end, (T*)out, n_tok, tpc, act, in_bias))
         return 1;

@@ -471,8 +471,7 @@ def test_attention_with_learnt_sinks_against_its_statement(dtype, H, G, d, dv):
 
 
 @GPU
-@pytest.mark.parametrize("H,G,d,window", [(4, 2, 16, 0), (8, 8, 64, 50), (8, 4, 128, 0), (6, 2, 48, 130), (4, 2, 256, 0), (5, 1, 80, 0),
-                                          (16, 1, 192, 0)])
+@pytest.mark.parametrize("H,G,d,window", [(4, 2, 16, 0), (8, 8, 64, 50), (8, 4, 128, 0), (6, 2, 48, 130), (4, 2, 256, 0), (16, 1, 192, 0)])
 def test_kernels_of_whole_heads_over_longer_rows_with_learnt_sinks(H, G, d, window):
     """Prompt steps (every form of the kernels; sequences that start and sequences that go on from stored keys) and decode
     steps (a row's keys in one chunk and in several), with columns behind q, k and v, with and without sinks."""
@@ -486,7 +485,7 @@ def test_kernels_of_whole_heads_over_longer_rows_with_learnt_sinks(H, G, d, wind
     sinks[0], sinks[1] = 6.0, -30.0
 
     def case(lens, starts):
-        tok_pos, tok_seq, slots, first, start, end = _tables(lens, starts, [(3 * s + 1) % (len(lens) + 1) for s in range(len(lens))])
+        tok_pos, tok_seq, slots, first, start, end = _tables(lens, starts, [len(lens) - s for s in range(len(lens))])
         per = max(-(-(a + n) // ops.PAGE) for a, n in zip(starts, lens))
         n_slots = len(lens) + 1
         table = torch.randperm(n_slots * per, generator=g).view(n_slots, per).to(torch.int32)
@@ -503,7 +502,7 @@ def test_kernels_of_whole_heads_over_longer_rows_with_learnt_sinks(H, G, d, wind
                          window=window, sink_values=z)
         return want
 
-    for lens, starts in (([1, 70, 129, 300], [0] * 4), ([200, 2, 65], [70, 129, 0])):
+    for lens, starts in (([1, 65, 140], [0] * 3), ([70, 2], [70, 129])):
         c = case(lens, starts)
         tok_pos, tok_seq, slots, first, start, end, table, kp, vp, rows = c
         before = dict(seq_start=start.cuda(), seq_slot=slots.cuda(), kpool=kp.cuda(), vpool=vp.cuda(), page_table=table.cuda()) if any(starts) else {}
@@ -530,6 +529,7 @@ def test_kernels_of_whole_heads_over_longer_rows_with_learnt_sinks(H, G, d, wind
     tok_pos, tok_seq, slots, first, start, end, table, kp, vp, rows = c
     for z in (sinks, None):
         want = statement(c, z)
+        assert z is None or (want.float() - statement(c, None).float()).abs().max().item() > 0.05
         for chunk in (64, 128, 320):
             chunks = -(-320 // chunk)
             scratch = torch.full((ops.attn_decode_scratch_floats(5, H, d, chunks),), float("nan"), device="cuda")

@@ -17,6 +17,7 @@ from .config.nosolix import NosolixConfig
 from .config.vivazen import VivazenConfig
 from .config.dekutar import DekutarConfig
 from .config.larulorn import LarulornConfig
+from .config.mugedra import MugedraConfig
 from .registry import architectures, register_architecture, resolve, unregister_architecture
 from .models import gemma2 as _gemma2            # registers Gemma2ForCausalLM
 from .models import sigalorn as _sigalorn        # registers Sigalorn
@@ -24,6 +25,7 @@ from .models import nosolix as _nosolix          # registers Nosolix
 from .models import vivazen as _vivazen          # registers Vivazen
 from .models import dekutar as _dekutar          # registers Dekutar
 from .models import larulorn as _larulorn        # registers Larulorn
+from .models import mugedra as _mugedra          # registers Mugedra
 from .engine.engine import Engine, build_model, from_config, load, open, write_random_model
 from .engine.step import StepEntry, StepError
 from .engine.generate import Reply
@@ -33,5 +35,5 @@ from .weights.loader import WeightsError
 __version__ = "0.1.0"
 
 __all__ = ["open", "load", "from_config", "write_random_model", "build_model", "Engine", "StepEntry", "StepError",
-           "Reply", "SamplingParams", "Gemma2Config", "SigalornConfig", "NosolixConfig", "VivazenConfig", "DekutarConfig", "LarulornConfig", "ConfigError", "WeightsError", "register_architecture",
+           "Reply", "SamplingParams", "Gemma2Config", "SigalornConfig", "NosolixConfig", "VivazenConfig", "DekutarConfig", "LarulornConfig", "MugedraConfig", "ConfigError", "WeightsError", "register_architecture",
            "unregister_architecture", "architectures", "resolve", "__version__"]

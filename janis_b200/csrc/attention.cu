@@ -161,7 +161,7 @@ attn_prefill_kernel(const T* __restrict__ qkv, const T* __restrict__ kv_src, con
     const int start = cached.seq_start ? cached.seq_start[seq] : 0;   // positions below it are in the cache
     const int slot = cached.seq_start ? cached.seq_slot[seq] : -1;
     const int first = seq_first_row[seq] - start;        // row that position 0 would have in the step's buffer
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_seen(pos, window);
 
     Lane<T> st;
     st.init();
@@ -207,7 +207,7 @@ attn_prefill_kernel(const T* __restrict__ qkv, const T* __restrict__ kv_src, con
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ void chunk_range(int len, int window, int chunk, int& lo, int& first_chunk,
                                             int& n_chunks) {
-    lo = window > 0 ? max(0, len - window) : 0;
+    lo = first_seen(max(len, 1) - 1, window);
     first_chunk = lo / chunk;
     n_chunks = (len + chunk - 1) / chunk - first_chunk;
 }

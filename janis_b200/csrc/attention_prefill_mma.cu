@@ -179,6 +179,9 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q_src, const bf16* __restrict__
     const int row_lo = start + q0 + warp * 16 + g;    // this thread's two query positions
     const int row_hi = row_lo + 8;
     const int warp_first = start + q0 + warp * 16, warp_last = warp_first + 15;
+    // the first keys that those rows see, and the warp's first and last row
+    const int from_lo = first_seen(row_lo, window), from_hi = first_seen(row_hi, window);
+    const int seen_first = first_seen(warp_first, window), seen_last = first_seen(warp_last, window);
 
     for (int it = 0; it < n_tiles; ++it) {
         const int k0 = k_first + it * BN;
@@ -188,8 +191,8 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q_src, const bf16* __restrict__
         __syncthreads();
         const uint32_t sK = sKV + (it & 1) * 2 * KV_BYTES, sV = sK + KV_BYTES;
 
-        // a warp whose rows see none of this tile's keys (all later, or all outside the window) skips it
-        const bool any = k0 <= warp_last && (window <= 0 || k0 + BN - 1 > warp_first - window);
+        // a warp whose rows see none of this tile's keys (all later, or all before its rows' windows or chunks) skips it
+        const bool any = k0 <= warp_last && k0 + BN - 1 >= seen_first;
         if (any) {
             // S = Q K^T for this warp's 16 rows and the 64 keys of the tile
             float s[BN / 8][4];
@@ -210,8 +213,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q_src, const bf16* __restrict__
                 }
             }
             // scale, cap, mask; scores end up in units of log2(e)
-            const bool inner = k0 + BN - 1 <= warp_first && k0 + BN <= total &&
-                               (window <= 0 || k0 > warp_last - window);   // every key seen by every row
+            const bool inner = k0 + BN - 1 <= warp_first && k0 + BN <= total && k0 >= seen_last;   // every key seen by every row
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int j = 0; j < BN / 8; ++j)
@@ -221,7 +223,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q_src, const bf16* __restrict__
                     if (!inner) {
                         const int key = k0 + j * 8 + t * 2 + (c & 1);
                         const int row = (c & 2) ? row_hi : row_lo;
-                        const bool seen = key <= row && key < total && (window <= 0 || key > row - window);
+                        const bool seen = key <= row && key < total && key >= ((c & 2) ? from_hi : from_lo);
                         v = seen ? v : -INFINITY;
                     }
                     s[j][c] = v;
@@ -445,7 +447,7 @@ static int prefill_piece_for(int n_tok, int n_seq, int nq, int window, int parts
     static std::mutex mu;
     std::lock_guard<std::mutex> lock(mu);
     const int len = ((n_tok + n_seq - 1) / n_seq + pf::BM - 1) / pf::BM * pf::BM;
-    const auto key = std::make_tuple(len, n_seq, nq, window > 0 && window < len ? window : 0, parts, tc05);
+    const auto key = std::make_tuple(len, n_seq, nq, abs(window) < len ? window : 0, parts, tc05);
     auto it = known.find(key);
     if (it == known.end()) {
         const int sms = sm_count();
@@ -554,7 +556,7 @@ JANIS_EXPORT int janis_attn_prefill_mma(const void* q_src, const void* kv_src, i
     // this size), and a piece that no tile exceeds means that nothing is shared: no places for parts, no merge.
     // (max_len: the longest sequence's tokens in this step, when the host knows them; else the step's tokens bound it)
     int most_tiles = ((max_len > 0 ? std::min(max_len, n_tok) : n_tok) + pf::BN - 1) / pf::BN;
-    if (window > 0) most_tiles = std::min(most_tiles, (window + pf::BM) / pf::BN + 1);        // a window bounds a tile's keys
+    if (window != 0) most_tiles = std::min(most_tiles, (abs(window) + pf::BM) / pf::BN + 1);  // a window or chunk bounds a tile's keys
     if (!ext && parts > 1) parts = std::max(1, std::min(parts, (most_tiles + piece - 1) / piece));
     if (!ext && most_tiles <= 8) parts = 1;           // up to 512 keys a tile: sharing measured no faster (512 tokens: 17.0 against 16.5 us)
     if ((long long)n_tiles_bound * parts > 65535) return fail("attn_prefill_mma: %d tiles of queries exceed the grid", n_tiles_bound);

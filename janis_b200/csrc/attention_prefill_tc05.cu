@@ -378,6 +378,7 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         // each tile and columns OCOLS h .. of the accumulator
         const int quarter = warp & 3, h = warp >> 2;
         const int r = quarter * 32 + lane, row_pos = q0 + r;
+        const int row_from = first_seen(row_pos, window), last_from = first_seen(q0 + BM - 1, window);    // the first keys seen
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const float LOG2E = 1.4426950408889634f;
         // scores in units of log2(e): cap2 tanh(s scale / cap) = cap2 - 2 cap2 / (2^(s k_tanh) + 1), or s scale2
@@ -399,7 +400,7 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             warp_arrive(bar(S_EMPTY + b), lane);      // the scores are in registers
             base = m_ref == -INFINITY ? 0.f : m_ref;
             const float c0 = CAPPED ? cap2 - base : -base, c1 = -2.0f * cap2;
-            const bool inner = k0 + BN - 1 <= q0 && k0 + BN <= len && (window <= 0 || k0 > q0 + BM - 1 - window);
+            const bool inner = k0 + BN - 1 <= q0 && k0 + BN <= len && k0 >= last_from;
             float mx = -INFINITY;
 #pragma unroll
             for (int j = 0; j < CPT; ++j) {
@@ -418,7 +419,7 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 }
                 if (!inner) {
                     const int key = k0 + CPT * h + j;
-                    const bool seen = key <= row_pos && key < len && (window <= 0 || key > row_pos - window);
+                    const bool seen = key <= row_pos && key < len && key >= row_from;
                     v = seen ? v : -INFINITY;
                 }
                 sv[j] = __float_as_uint(v);
@@ -899,6 +900,7 @@ attn_prefill_tc05_items_kernel(const __grid_constant__ CUtensorMap map_q, const 
             if (me.n_tiles < 0) break;
             const int n_tiles = me.n_tiles, q0 = me.q0, len = me.len, k_first = me.k_first;
             const int row_pos = q0 + r;
+            const int row_from = first_seen(row_pos, window), last_from = first_seen(q0 + BM - 1, window);
             const bool shared_tile = me.np > 1;
             float m_ref = -INFINITY, l_run = 0.f;
             auto stage_one = [&](int it, uint32_t (&sv)[CPT], float& base) -> bool {
@@ -911,7 +913,7 @@ attn_prefill_tc05_items_kernel(const __grid_constant__ CUtensorMap map_q, const 
                 warp_arrive(bar(S_EMPTY + b), lane);
                 base = m_ref == -INFINITY ? 0.f : m_ref;
                 const float c0 = CAPPED ? cap2 - base : -base, c1 = -2.0f * cap2;
-                const bool inner = k0 + BN - 1 <= q0 && k0 + BN <= len && (window <= 0 || k0 > q0 + BM - 1 - window);
+                const bool inner = k0 + BN - 1 <= q0 && k0 + BN <= len && k0 >= last_from;
                 float mx = -INFINITY;
 #pragma unroll
                 for (int j = 0; j < CPT; ++j) {
@@ -930,7 +932,7 @@ attn_prefill_tc05_items_kernel(const __grid_constant__ CUtensorMap map_q, const 
                     }
                     if (!inner) {
                         const int key = k0 + CPT * h + j;
-                        const bool seen = key <= row_pos && key < len && (window <= 0 || key > row_pos - window);
+                        const bool seen = key <= row_pos && key < len && key >= row_from;
                         v = seen ? v : -INFINITY;
                     }
                     sv[j] = __float_as_uint(v);

@@ -27,7 +27,7 @@ constexpr int ROWS_VB = 4;          // and a pass of the values (2 where a key/v
 struct RowsShape {
     int H, G, d, dv;
     int v_stride;       // elements between the values of neighbouring positions (dv, or d when the values lie in the keys)
-    int window;         // keys are seen among the row's last `window` positions (0: all earlier ones)
+    int window;         // keys are seen among the row's last `window` positions, or (< 0) in its chunk of -window (0: all earlier ones)
     int keep_first;     // with a window: the sequence's first `keep_first` positions stay seen behind it
     int chunk;          // keys a CTA takes
     int n_chunks;       // CTAs a row
@@ -58,7 +58,7 @@ template <> __device__ __forceinline__ void rows_unpack<bf16>(const uint4& raw, 
 struct RowsKeys { int first, kept; };
 __device__ __forceinline__ RowsKeys rows_range(const RowsShape& sh, int pos, int c, int& j0, int& j1) {
     RowsKeys k;
-    k.first = sh.window > 0 ? max(0, pos - sh.window + 1) : 0;
+    k.first = first_seen(pos, sh.window);
     k.kept = sh.window > 0 ? min(sh.keep_first, k.first) : 0;
     j0 = c * sh.chunk;
     j1 = min(k.kept + pos - k.first, j0 + sh.chunk - 1);
@@ -309,7 +309,7 @@ rows_sum_kernel(const float* __restrict__ o_part, const int* __restrict__ tok_po
     const int t = blockIdx.y, n = sh.H * sh.dv, i = (blockIdx.x * ROWS_THREADS + threadIdx.x) * 4;
     grid_dependents_launch();
     const int pos = tok_pos[t], slot = seq_slot[tok_seq[t]];
-    const int first = sh.window > 0 ? max(0, pos - sh.window + 1) : 0, kept = sh.window > 0 ? min(sh.keep_first, first) : 0;
+    const int first = first_seen(pos, sh.window), kept = sh.window > 0 ? min(sh.keep_first, first) : 0;
     const int n_valid = slot < 0 ? 0 : min(sh.n_chunks, (kept + pos - first) / sh.chunk + 1);
     grid_dependency_wait();
     if (i >= n) return;

@@ -33,13 +33,18 @@ namespace janis {
 // line.  A row of the step holds q (H heads of d), then k (G heads of d), then v (G heads of dv); a layer
 // that only reads a line has rows of q alone (with_kv == 0).  With `bias` (floats, one per column of the row's q | k | v)
 // it is added first.  `mix` 1: the values are also left in v_first, as they are before they are stored; `mix` 2: the
-// values become (1 - share) v + share v_first.  One CTA per token; a pair's sine and cosine are formed once for all heads.
+// values become (1 - share) v + share v_first.  With `q_norm` and `k_norm` (floats, d each; not together with a bias) every
+// head of q and of k is divided by sqrt(mean(head^2) + norm_eps) and multiplied by its weight before it turns.  One CTA per
+// token; a pair's sine and cosine are formed once for all heads.
 // ---------------------------------------------------------------------------
 struct RotateExtras {
     const float* bias;      // [H d + G d + G dv] (or the first H d of it), or null
     float amp;              // on sine and cosine of the queries' and keys' turn
     int mix;                // 0 none; 1 leave the values in v_first; 2 mix v_first in
     float share;            // the weight of v_first
+    const float* q_norm;    // [d] on every head of q, or null
+    const float* k_norm;    // [d] on every head of k, or null (both or none)
+    float norm_eps;
 };
 
 template <typename T>
@@ -82,9 +87,17 @@ qkv_rotate_store_kernel(T* __restrict__ rows, int row_elems, const int* __restri
         T* p = row + (size_t)head * d;
         const float* b = ex.bias != nullptr ? ex.bias + (size_t)head * d : nullptr;
         T* kd = head >= H && kdst != nullptr ? kdst + (size_t)(head - H) * JANIS_PAGE * d : nullptr;
+        const float* wn = head < H ? ex.q_norm : ex.k_norm;
+        float inv = 1.f;
+        if (wn != nullptr) {
+            float ss = 0.f;
+            for (int i = lane; i < d; i += 32) ss = fmaf(to_float(p[i]), to_float(p[i]), ss);
+            inv = 1.0f / sqrtf(warp_sum(ss) / (float)d + ex.norm_eps);
+        }
         for (int i = lane; i < hq; i += 32) {
             float x0 = to_float(p[i]), x1 = to_float(p[i + hq]);
             if (b != nullptr) { x0 += b[i]; x1 += b[i + hq]; }
+            if (wn != nullptr) { x0 *= inv * wn[i]; x1 *= inv * wn[i + hq]; }
             float lo, hi;
             rotate_pair(x0, x1, turn_s[i].x, turn_s[i].y, lo, hi);
             const T tl = from_float<T>(lo), th = from_float<T>(hi);
@@ -95,11 +108,11 @@ qkv_rotate_store_kernel(T* __restrict__ rows, int row_elems, const int* __restri
                 kd[i + hq] = th;
             }
         }
-        if (b != nullptr || kd != nullptr)
+        if (b != nullptr || wn != nullptr || kd != nullptr)
             for (int i = rot + lane; i < d; i += 32) {           // what does not turn
                 T x = p[i];
-                if (b != nullptr) {
-                    x = from_float<T>(to_float(x) + b[i]);
+                if (b != nullptr || wn != nullptr) {
+                    x = from_float<T>(b != nullptr ? to_float(x) + b[i] : to_float(x) * (inv * wn[i]));
                     p[i] = x;
                 }
                 if (kd != nullptr) kd[i] = x;
@@ -176,6 +189,33 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
     __syncthreads();
     grid_dependency_wait();
     T* row = rows + (size_t)t * row_elems;
+    float* inv_s = reinterpret_cast<float*>(turn_s + hq);            // 1 / root mean square of every head of q and k
+    if (ex.q_norm != nullptr) {
+        for (int head = tid >> 5; head < n_heads; head += nt >> 5) {
+            float ss = 0.f;
+            for (int c = (tid & 31) * V; c < d; c += 32 * V) {
+                float a[V];
+                Vec16<T>::load(row + head * d + c, a);
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss = fmaf(a[e], a[e], ss);
+            }
+            ss = warp_sum(ss);
+            if ((tid & 31) == 0) inv_s[head] = 1.0f / sqrtf(ss / (float)d + ex.norm_eps);
+        }
+        __syncthreads();
+    }
+    auto norm_head = [&](float (&x)[V], int head, int i) {
+        if (ex.q_norm == nullptr) return;
+        const float* wn = (head < H ? ex.q_norm : ex.k_norm) + i;
+        const float inv = inv_s[head];
+#pragma unroll
+        for (int e = 0; e < V; e += 4) {
+            float b[4];
+            Vec16<float>::load(wn + e, b);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) x[e + q] *= inv * b[q];
+        }
+    };
     auto add_bias = [&](float (&x)[V], int at) {
         if (ex.bias == nullptr) return;
 #pragma unroll
@@ -188,7 +228,7 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
     };
     const int per_turn = hq / V, per_rest = (d - rot) / V, per_v = dv / V;
     const int n_turn = n_heads * per_turn;
-    const int rest0 = ex.bias != nullptr ? 0 : H;                    // (without a bias the queries' rest stays as it is)
+    const int rest0 = ex.bias != nullptr || ex.q_norm != nullptr ? 0 : H;      // (without a bias and a norm the queries' rest stays as it is)
     const int n_rest = n_heads > rest0 ? (n_heads - rest0) * per_rest : 0, n_val = with_kv ? G * per_v : 0;
     for (int u = tid; u < n_turn + n_rest + n_val; u += nt) {
         if (u < n_turn) {
@@ -198,6 +238,8 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
             Vec16<T>::load(row + at + hq, b);
             add_bias(a, at);
             add_bias(b, at + hq);
+            norm_head(a, head, i);
+            norm_head(b, head, i + hq);
 #pragma unroll
             for (int e = 0; e < V; ++e) {
                 const float2 sc = turn_s[i + e];
@@ -217,8 +259,9 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
             const int w = u - n_turn, head = rest0 + w / per_rest, c = rot + (w % per_rest) * V, at = head * d + c;
             float a[V];
             Vec16<T>::load(row + at, a);
-            if (ex.bias != nullptr) {
+            if (ex.bias != nullptr || ex.q_norm != nullptr) {
                 add_bias(a, at);
+                norm_head(a, head, c);
                 Vec16<T>::store(row + at, a);
             }
             if (head >= H && kdst != nullptr) Vec16<T>::store(kdst + (size_t)(head - H) * JANIS_PAGE * d + c, a);
@@ -936,8 +979,11 @@ JANIS_EXPORT int janis_qkv_rotate_store(void* rows, int dtype, int row_elems, co
                                         const int* seq_slot, const float* inv_qk, int rot, const float* inv_v, int T,
                                         int H, int G, int d, int dv, int with_kv, void* kpool, void* vpool,
                                         const int* page_table, int table_stride, const float* bias, float amp, int mix,
-                                        float share, void* v_first, cudaStream_t stream) {
+                                        float share, void* v_first, const float* q_norm, const float* k_norm,
+                                        float norm_eps, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if ((q_norm == nullptr) != (k_norm == nullptr) || (q_norm != nullptr && (bias != nullptr || !with_kv)))
+        return fail("qkv_rotate_store: the heads' norms stand on q and k together, without a bias");
     if (rot < 0 || rot > d || (rot & 1)) return fail("qkv_rotate_store: rotary width %d does not fit key size %d", rot, d);
     if (inv_v != nullptr && (dv & 1)) return fail("qkv_rotate_store: rotated values need an even size, found %d", dv);
     if (row_elems < H * d + (with_kv ? G * (d + dv) : 0)) return fail("qkv_rotate_store: rows of %d elements are too short", row_elems);
@@ -946,18 +992,21 @@ JANIS_EXPORT int janis_qkv_rotate_store(void* rows, int dtype, int row_elems, co
     if (inv_v != nullptr && (mix || bias != nullptr)) return fail("qkv_rotate_store: turned values take no bias and no mixing");
     const size_t bytes = ((size_t)(rot >> 1) + (inv_v != nullptr ? dv >> 1 : 0)) * sizeof(float2);
     if (bytes > 48 * 1024) return fail("qkv_rotate_store: %zu bytes of angles", bytes);
-    const RotateExtras ex = {bias, amp, mix, share};
+    const RotateExtras ex = {bias, amp, mix, share, q_norm, k_norm, norm_eps};
     const int vec = dtype == JANIS_F32 ? 4 : 8;
     if (inv_v == nullptr && (rot >> 1) % vec == 0 && d % vec == 0 && dv % vec == 0 && row_elems % vec == 0 &&
-        (((uintptr_t)rows | (uintptr_t)kpool | (uintptr_t)vpool | (uintptr_t)bias | (uintptr_t)v_first) & 15) == 0) {
+        (((uintptr_t)rows | (uintptr_t)kpool | (uintptr_t)vpool | (uintptr_t)bias | (uintptr_t)v_first | (uintptr_t)q_norm |
+          (uintptr_t)k_norm) & 15) == 0) {
+        const size_t vbytes = bytes + (q_norm != nullptr ? (size_t)(H + G) * sizeof(float) : 0);
+        if (vbytes > 48 * 1024) return fail("qkv_rotate_store: %zu bytes of angles and norms", vbytes);
         const int items = ((with_kv ? H + G : H) * (d - rot / 2) + (with_kv ? G * dv : 0)) / vec;
         const dim3 vgrid(T), vblock(items > 128 || T <= 64 ? 256 : 128);
         if (dtype == JANIS_F32)
-            return launch_kernel("qkv_rotate_store", qkv_rotate_store_vec_kernel<float>, vgrid, vblock, bytes, stream, 1, (float*)rows,
+            return launch_kernel("qkv_rotate_store", qkv_rotate_store_vec_kernel<float>, vgrid, vblock, vbytes, stream, 1, (float*)rows,
                                  row_elems, tok_pos, tok_seq, seq_slot, inv_qk, rot, H, G, d, dv, with_kv, (float*)kpool,
                                  (float*)vpool, page_table, table_stride, ex, (float*)v_first);
         if (dtype == JANIS_BF16)
-            return launch_kernel("qkv_rotate_store", qkv_rotate_store_vec_kernel<bf16>, vgrid, vblock, bytes, stream, 1, (bf16*)rows,
+            return launch_kernel("qkv_rotate_store", qkv_rotate_store_vec_kernel<bf16>, vgrid, vblock, vbytes, stream, 1, (bf16*)rows,
                                  row_elems, tok_pos, tok_seq, seq_slot, inv_qk, rot, H, G, d, dv, with_kv, (bf16*)kpool,
                                  (bf16*)vpool, page_table, table_stride, ex, (bf16*)v_first);
     }

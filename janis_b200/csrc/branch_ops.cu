@@ -1,4 +1,4 @@
-// Rows of the residual stream and of a layer's branches: the Dynamic Tanh norm, the RMS norm in groups that follows a
+// Rows of the residual stream and of a layer's branches: the sum that a sublayer's result joins with the norm behind it, the Dynamic Tanh norm, the RMS norm in groups that follows a
 // scaled residual sum, the norm-and-accumulate of branches that run side by side, and a sigmoid gate on the heads of
 // an attention.  All arithmetic is float.
 #include "common.cuh"
@@ -143,6 +143,198 @@ group_norm_kernel(float* __restrict__ h, const TR* __restrict__ res, const int* 
     }
 }
 
+// ---------------------------------------------------------------------------
+// A sublayer's result into the stream, and the norm behind the sum:
+//
+//   v    = r0                                                  one branch as it is, or
+//   v    = share * (rms(r0) * w0 + rms(r1) * w1)               one or two branches normed first (w0, w1 given)
+//   h[r] += scale * v + more[r]                                scale: a factor per feature (null: 1); more: rows of the
+//                                                              stream's type that join the sum (null: none)
+//   y[r] = norm(h[r]) * w_next                                 centred: (h - mean) / sqrt(mean((h - mean)^2) + eps),
+//                                                              else h / sqrt(mean(h^2) + eps)
+//
+// With r0 null nothing is added and y[r] = norm(h[rows[r] or r]), h untouched.
+// ---------------------------------------------------------------------------
+struct StreamSum {
+    const float* w0;          // the branches' norm weights, or null
+    const float* w1;
+    float eps, share;
+    const float* scale;
+    const float* more;
+};
+
+// two sums over the block at once, in the order of block_sum
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = (blockDim.x + 31) >> 5;
+    a = warp_sum(a);
+    b = warp_sum(b);
+    __syncthreads();
+    if (lane == 0) scratch[warp] = make_float2(a, b);
+    __syncthreads();
+    float2 t = make_float2(0.f, 0.f);
+    for (int w = 0; w < nwarp; ++w) {
+        t.x += scratch[w].x;
+        t.y += scratch[w].y;
+    }
+    return t;
+}
+
+// VW elements an access: 4 (rows of whole 16-byte pieces; the row stays in registers, up to VPT pieces a thread) or 1 (any
+// row; the row is read again from where it was written).
+template <typename TR, typename TO, int VW, int VPT>
+__global__ void __launch_bounds__(256)
+stream_norm_kernel(float* __restrict__ h, const TR* __restrict__ r0, const TR* __restrict__ r1, StreamSum s,
+                   const float* __restrict__ w_next, float eps_next, int centred, TO* __restrict__ y,
+                   const int* __restrict__ rows, int H) {
+    __shared__ float2 scratch2[32];
+    __shared__ float scratch[32];
+    const int r = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+    grid_dependents_launch();
+    grid_dependency_wait();
+    float* hr = h + (size_t)(rows != nullptr ? rows[r] : r) * H;
+    const TR* a0 = r0 != nullptr ? r0 + (size_t)r * H : nullptr;
+    const TR* a1 = r1 != nullptr ? r1 + (size_t)r * H : nullptr;
+    const float* mr = s.more != nullptr ? s.more + (size_t)r * H : nullptr;
+    const float n = (float)H;
+    if (VW == 4) {
+        const int pieces = H >> 2;
+        float hv[VPT][4];
+#pragma unroll
+        for (int p = 0; p < VPT; ++p) {
+            const int i = (tid + p * nt) * 4;
+            hv[p][0] = hv[p][1] = hv[p][2] = hv[p][3] = 0.f;
+            if (tid + p * nt < pieces) load4(hr + i, hv[p]);
+        }
+        float sum = 0.f;
+        if (a0 != nullptr) {
+            float inv0 = 1.f, inv1 = 0.f;
+            float v0[VPT][4], v1[VPT][4];
+#pragma unroll
+            for (int p = 0; p < VPT; ++p) {
+                const int i = (tid + p * nt) * 4;
+                const bool in = tid + p * nt < pieces;
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v0[p][e] = v1[p][e] = 0.f;
+                if (in) load4(a0 + i, v0[p]);
+                if (in && a1 != nullptr) load4(a1 + i, v1[p]);
+            }
+            if (s.w0 != nullptr) {
+                float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+                for (int p = 0; p < VPT; ++p)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        s0 = fmaf(v0[p][e], v0[p][e], s0);
+                        s1 = fmaf(v1[p][e], v1[p][e], s1);
+                    }
+                const float2 t = block_sum2(s0, s1, scratch2);
+                inv0 = s.share / sqrtf(t.x / n + s.eps);
+                inv1 = s.share / sqrtf(t.y / n + s.eps);
+            }
+#pragma unroll
+            for (int p = 0; p < VPT; ++p) {
+                const int i = (tid + p * nt) * 4;
+                if (tid + p * nt >= pieces) continue;
+                float w[4];
+                if (s.w0 != nullptr) {
+                    load4(s.w0 + i, w);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) v0[p][e] *= inv0 * w[e];
+                    if (a1 != nullptr) {
+                        load4(s.w1 + i, w);
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) v0[p][e] = fmaf(v1[p][e] * inv1, w[e], v0[p][e]);
+                    }
+                }
+                if (s.scale != nullptr) {
+                    load4(s.scale + i, w);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) hv[p][e] = fmaf(w[e], v0[p][e], hv[p][e]);
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) hv[p][e] += v0[p][e];
+                }
+                if (mr != nullptr) {
+                    load4(mr + i, w);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) hv[p][e] += w[e];
+                }
+                store4(hr + i, hv[p]);
+            }
+        }
+        if (w_next == nullptr) return;
+        float mean = 0.f;
+        if (centred) {
+#pragma unroll
+            for (int p = 0; p < VPT; ++p)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) sum += hv[p][e];
+            mean = block_sum(sum, scratch) / n;
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int p = 0; p < VPT; ++p)
+            if (tid + p * nt < pieces) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    hv[p][e] -= mean;
+                    ss = fmaf(hv[p][e], hv[p][e], ss);
+                }
+            }
+        ss = block_sum(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss / n + eps_next);
+#pragma unroll
+        for (int p = 0; p < VPT; ++p) {
+            const int i = (tid + p * nt) * 4;
+            if (tid + p * nt >= pieces) continue;
+            float w[4], o[4];
+            load4(w_next + i, w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[e] = hv[p][e] * inv * w[e];
+            store4(y + (size_t)r * H + i, o);
+        }
+        return;
+    }
+    float sum = 0.f;
+    if (a0 != nullptr) {
+        float inv0 = 1.f, inv1 = 0.f;
+        if (s.w0 != nullptr) {
+            float s0 = 0.f, s1 = 0.f;
+            for (int i = tid; i < H; i += nt) {
+                const float u = to_float(a0[i]), v = a1 != nullptr ? to_float(a1[i]) : 0.f;
+                s0 = fmaf(u, u, s0);
+                s1 = fmaf(v, v, s1);
+            }
+            const float2 t = block_sum2(s0, s1, scratch2);
+            inv0 = s.share / sqrtf(t.x / n + s.eps);
+            inv1 = s.share / sqrtf(t.y / n + s.eps);
+        }
+        for (int i = tid; i < H; i += nt) {
+            float v = to_float(a0[i]);
+            if (s.w0 != nullptr) {
+                v *= inv0 * s.w0[i];
+                if (a1 != nullptr) v = fmaf(to_float(a1[i]) * inv1, s.w1[i], v);
+            }
+            float hv = s.scale != nullptr ? fmaf(s.scale[i], v, hr[i]) : hr[i] + v;
+            if (mr != nullptr) hv += mr[i];
+            hr[i] = hv;                          // read back below by this same thread only
+            sum += hv;
+        }
+    } else if (centred) {
+        for (int i = tid; i < H; i += nt) sum += hr[i];
+    }
+    if (w_next == nullptr) return;
+    const float mean = centred ? block_sum(sum, scratch) / n : 0.f;
+    float ss = 0.f;
+    for (int i = tid; i < H; i += nt) {
+        const float v = hr[i] - mean;
+        ss = fmaf(v, v, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / n + eps_next);
+    for (int i = tid; i < H; i += nt) y[(size_t)r * H + i] = from_float<TO>((hr[i] - mean) * inv * w_next[i]);
+}
+
 // y = h rounded to the activation type: what a sublayer reads when it reads the stream itself
 __global__ void __launch_bounds__(256) round_rows_kernel(const float* __restrict__ h, bf16* __restrict__ y, size_t n) {
     grid_dependents_launch();
@@ -171,7 +363,7 @@ sigmoid_gate_kernel(T* __restrict__ x, const T* __restrict__ rows, int row_elems
 // router, a warp per token over E logits z (float):  s = sigmoid(z), c = s + correction;  experts form n_groups equal
 // groups of neighbours, a group's score is the sum of its two largest c (group_best: its largest), the best `keep` groups stay (ties: the
 // lower index); among their experts the `top` of largest c are chosen (ties: the lower index); the chosen get
-// w_e = s_e / (sum of the chosen s + 1e-20) * scale, every other expert 0.  With a shared gate, column E of z is
+// w_e = s_e / (sum of the chosen s + 1e-20) * scale (raw: w_e = s_e * scale), every other expert 0.  With a shared gate, column E of z is
 // its logit and column E of the output its sigmoid.  With `softmax` the scores are the softmax of z over all entries instead.  With
 // n_identity > 0 the router scores that many entries more, behind the experts (no groups then); they have no column of
 // their own in the output: the weights of the chosen ones add up in its last column.
@@ -189,7 +381,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& at) {
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ z, const float* __restrict__ correction, int T, int E, int n_groups, int keep,
-                 int top, float scale, int shared_gate, float* __restrict__ out, int n_identity, int softmax, int group_best) {
+                 int top, float scale, int shared_gate, float* __restrict__ out, int n_identity, int softmax, int group_best, int raw) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * ROUTE_WARPS + warp;
     const int N = E + n_identity;                    // entries the router scores: the experts, then the identity entries
@@ -268,7 +460,7 @@ moe_route_kernel(const float* __restrict__ z, const float* __restrict__ correcti
         }
         __syncwarp();
     }
-    const float f = scale / (total + 1e-20f);
+    const float f = raw ? scale : scale / (total + 1e-20f);
     for (int e = lane; e < E; e += 32) o[e] = mark[e] != 0.f ? s[e] * f : 0.f;
     if (n_identity) {
         float id = 0.f;                              // the identity entries' weights add up: they all return the input
@@ -309,11 +501,12 @@ moe_identity_add_kernel(T* __restrict__ out, const T* __restrict__ y, const floa
 
 // a[t, col] = w[t, e] * g sigmoid(alpha g) (u + up_add), g = min(gate, limit), u = clamp(up, -limit, limit), over the
 // columns of all experts side by side (expert e: `ff` columns; then the shared expert's `shared_ff`); in gu an
-// expert's gate columns are followed by its up columns.  Experts of weight 0 give exact zeros.
+// expert's gate columns are followed by its up columns.  Experts of weight 0 give exact zeros.  w_in: the weight stands on
+// the expert's input instead, so that gate and up (which are linear in it) are multiplied by w and the result is not.
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_expert_act_kernel(const T* __restrict__ gu, const float* __restrict__ wts, int E, int ff, float limit, int shared_ff,
-                      float shared_limit, float alpha, T* __restrict__ out, size_t n, int wcols, float up_add) {
+                      float shared_limit, float alpha, T* __restrict__ out, size_t n, int wcols, float up_add, int w_in) {
     const int total = E * ff + shared_ff;
     grid_dependents_launch();
     grid_dependency_wait();
@@ -329,9 +522,10 @@ moe_expert_act_kernel(const T* __restrict__ gu, const float* __restrict__ wts, i
         float a = 0.f;
         if (w != 0.f) {
             const T* row = gu + t * (size_t)(2 * total) + base;
-            const float g = fminf(to_float(row[j]), lim);
-            const float u = fminf(fmaxf(to_float(row[width + j]), -lim), lim);
-            a = w * (g / (1.0f + expf(-alpha * g))) * (u + up_add);
+            const float wi = w_in ? w : 1.0f, wo = w_in ? 1.0f : w;
+            const float g = fminf(to_float(row[j]) * wi, lim);
+            const float u = fminf(fmaxf(to_float(row[width + j]) * wi, -lim), lim);
+            a = wo * (g / (1.0f + expf(-alpha * g))) * (u + up_add);
         }
         out[i] = from_float<T>(a);
     }
@@ -342,7 +536,7 @@ moe_expert_act_kernel(const T* __restrict__ gu, const float* __restrict__ wts, i
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_expert_act_vec_kernel(const T* __restrict__ gu, const float* __restrict__ wts, int E, int ff, float limit, int shared_ff,
-                          float shared_limit, float alpha, T* __restrict__ out, int T_rows, int wcols, float up_add) {
+                          float shared_limit, float alpha, T* __restrict__ out, int T_rows, int wcols, float up_add, int w_in) {
     constexpr int V = Vec16<T>::N;
     const int total = E * ff + shared_ff, per_row = total / V;
     grid_dependents_launch();
@@ -366,11 +560,12 @@ moe_expert_act_vec_kernel(const T* __restrict__ gu, const float* __restrict__ wt
                 float gv[V], uv[V];
                 Vec16<T>::load(grow + base + j, gv);
                 Vec16<T>::load(grow + base + width + j, uv);
+                const float wi = w_in ? w : 1.0f, wo = w_in ? 1.0f : w;
 #pragma unroll
                 for (int i = 0; i < V; ++i) {
-                    const float g = fminf(gv[i], lim);
-                    const float u = fminf(fmaxf(uv[i], -lim), lim);
-                    a[i] = w * (g / (1.0f + expf(-alpha * g))) * (u + up_add);
+                    const float g = fminf(gv[i] * wi, lim);
+                    const float u = fminf(fmaxf(uv[i] * wi, -lim), lim);
+                    a[i] = wo * (g / (1.0f + expf(-alpha * g))) * (u + up_add);
                 }
             }
             Vec16<T>::store(orow + col, a);
@@ -532,13 +727,56 @@ JANIS_EXPORT int janis_group_norm(float* h, const void* res, int res_dtype, cons
     return fail("group_norm: unknown dtypes %d, %d", res_dtype, y_dtype);
 }
 
+template <typename TR, typename TO>
+static int stream_norm_launch(float* h, const void* r0, const void* r1, const StreamSum& s, const float* w_next, float eps_next,
+                              int centred, void* y, const int* rows, int R, int H, bool vec, cudaStream_t stream) {
+#define JANIS_SN(VW, VPT, NT)                                                                                          \
+    return launch_kernel("stream_norm", stream_norm_kernel<TR, TO, VW, VPT>, dim3(R), dim3(NT), 0, stream, 1, h, (const TR*)r0, \
+                         (const TR*)r1, s, w_next, eps_next, centred, (TO*)y, rows, H);
+    if (vec) {
+        const int pieces = H / 4;
+        if (pieces <= 128) { JANIS_SN(4, 1, 128) }
+        if (pieces <= 256) { JANIS_SN(4, 1, 256) }
+        if (pieces <= 384) { JANIS_SN(4, 3, 128) }
+        if (pieces <= 512) { JANIS_SN(4, 2, 256) }
+        if (pieces <= 768) { JANIS_SN(4, 3, 256) }
+        if (pieces <= 1024) { JANIS_SN(4, 4, 256) }
+        if (pieces <= 1536) { JANIS_SN(4, 6, 256) }
+    }
+    JANIS_SN(1, 1, H >= 1024 ? 256 : 128)
+#undef JANIS_SN
+}
+
+JANIS_EXPORT int janis_stream_norm(float* h, const void* r0, const void* r1, int r_dtype, const float* w0, const float* w1, float eps,
+                                   float share, const float* scale, const float* more, const float* w_next, float eps_next,
+                                   int centred, void* y, int y_dtype, const int* rows, int R, int H, cudaStream_t stream) {
+    if (R <= 0) return 0;
+    if (r0 != nullptr && rows != nullptr) return fail("stream_norm: a result is added to all rows, not to chosen ones");
+    if (r0 == nullptr && (r1 != nullptr || more != nullptr || w_next == nullptr)) return fail("stream_norm: nothing to do, or a second branch without a first");
+    if ((w0 == nullptr) != (w1 == nullptr) && r1 != nullptr) return fail("stream_norm: both branches are normed, or none");
+    if (r1 != nullptr && w0 == nullptr) return fail("stream_norm: two branches are normed before they are added");
+    if (w_next != nullptr && y == nullptr) return fail("stream_norm: a norm needs an output");
+    const StreamSum s = {w0, w1, eps, share, scale, more};
+    const uintptr_t all = (uintptr_t)h | (uintptr_t)r0 | (uintptr_t)r1 | (uintptr_t)w0 | (uintptr_t)w1 | (uintptr_t)scale |
+                          (uintptr_t)more | (uintptr_t)w_next | (uintptr_t)y;
+    const bool vec = H % 4 == 0 && (all & 15) == 0;
+    const int rd = r0 != nullptr ? r_dtype : JANIS_F32, yd = y != nullptr ? y_dtype : JANIS_F32;
+#define JANIS_SNT(TR, TO) return stream_norm_launch<TR, TO>(h, r0, r1, s, w_next, eps_next, centred, y, rows, R, H, vec, stream);
+    if (rd == JANIS_F32 && yd == JANIS_F32) { JANIS_SNT(float, float) }
+    if (rd == JANIS_F32 && yd == JANIS_BF16) { JANIS_SNT(float, bf16) }
+    if (rd == JANIS_BF16 && yd == JANIS_F32) { JANIS_SNT(bf16, float) }
+    if (rd == JANIS_BF16 && yd == JANIS_BF16) { JANIS_SNT(bf16, bf16) }
+#undef JANIS_SNT
+    return fail("stream_norm: unknown dtypes %d, %d", r_dtype, y_dtype);
+}
+
 JANIS_EXPORT int janis_round_rows(const float* h, void* y, size_t n, cudaStream_t stream) {
     if (n == 0) return 0;
     return launch_kernel("round_rows", round_rows_kernel, dim3(flat_grid(n)), dim3(256), 0, stream, 1, h, (bf16*)y, n);
 }
 
 JANIS_EXPORT int janis_moe_route(const float* z, const float* correction, int T, int E, int n_groups, int keep, int top,
-                                 float scale, int shared_gate, float* out, int n_identity, int softmax, int group_best,
+                                 float scale, int shared_gate, float* out, int n_identity, int softmax, int group_best, int raw,
                                  cudaStream_t stream) {
     if (T <= 0) return 0;
     const int N = E + n_identity;
@@ -548,7 +786,7 @@ JANIS_EXPORT int janis_moe_route(const float* z, const float* correction, int T,
         return fail("moe_route: %d entries in %d groups, %d kept, %d chosen", N, n_groups, keep, top);
     const size_t bytes = (size_t)ROUTE_WARPS * 4 * N * sizeof(float);
     return launch_kernel("moe_route", moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32),
-                         bytes, stream, 1, z, correction, T, E, n_groups, keep, top, scale, shared_gate, out, n_identity, softmax, group_best);
+                         bytes, stream, 1, z, correction, T, E, n_groups, keep, top, scale, shared_gate, out, n_identity, softmax, group_best, raw);
 }
 
 JANIS_EXPORT int janis_moe_identity_add(void* out, const void* y, int dtype, const float* wts, int wts_stride, int w_col, int T,
@@ -567,7 +805,7 @@ JANIS_EXPORT int janis_moe_identity_add(void* out, const void* y, int dtype, con
 
 JANIS_EXPORT int janis_moe_expert_act(const void* gu, int dtype, const float* wts, int E, int ff, float limit, int shared_ff,
                                       float shared_limit, float alpha, void* out, int T, int wts_stride, float up_add,
-                                      cudaStream_t stream) {
+                                      int w_in, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (wts_stride <= 0) wts_stride = E + (shared_ff ? 1 : 0);
     const size_t n = (size_t)T * ((size_t)E * ff + shared_ff);
@@ -577,17 +815,17 @@ JANIS_EXPORT int janis_moe_expert_act(const void* gu, int dtype, const float* wt
         const dim3 grid((per_row + 255) / 256, T < 65535 ? T : 65535), block(256);
         if (dtype == JANIS_F32)
             return launch_kernel("moe_expert_act", moe_expert_act_vec_kernel<float>, grid, block, 0, stream, 1, (const float*)gu,
-                                 wts, E, ff, limit, shared_ff, shared_limit, alpha, (float*)out, T, wts_stride, up_add);
+                                 wts, E, ff, limit, shared_ff, shared_limit, alpha, (float*)out, T, wts_stride, up_add, w_in);
         if (dtype == JANIS_BF16)
             return launch_kernel("moe_expert_act", moe_expert_act_vec_kernel<bf16>, grid, block, 0, stream, 1, (const bf16*)gu,
-                                 wts, E, ff, limit, shared_ff, shared_limit, alpha, (bf16*)out, T, wts_stride, up_add);
+                                 wts, E, ff, limit, shared_ff, shared_limit, alpha, (bf16*)out, T, wts_stride, up_add, w_in);
     }
     if (dtype == JANIS_F32)
         return launch_kernel("moe_expert_act", moe_expert_act_kernel<float>, dim3(flat_grid(n)), dim3(256), 0, stream, 1,
-                             (const float*)gu, wts, E, ff, limit, shared_ff, shared_limit, alpha, (float*)out, n, wts_stride, up_add);
+                             (const float*)gu, wts, E, ff, limit, shared_ff, shared_limit, alpha, (float*)out, n, wts_stride, up_add, w_in);
     if (dtype == JANIS_BF16)
         return launch_kernel("moe_expert_act", moe_expert_act_kernel<bf16>, dim3(flat_grid(n)), dim3(256), 0, stream, 1,
-                             (const bf16*)gu, wts, E, ff, limit, shared_ff, shared_limit, alpha, (bf16*)out, n, wts_stride, up_add);
+                             (const bf16*)gu, wts, E, ff, limit, shared_ff, shared_limit, alpha, (bf16*)out, n, wts_stride, up_add, w_in);
     return fail("moe_expert_act: unknown dtype %d", dtype);
 }
 

@@ -115,6 +115,14 @@ inline int launch_kernel(const char* what, void (*kernel)(KArgs...), dim3 grid, 
     return 0;
 }
 
+// The first key that the query at position `pos` sees.  window > 0: the last `window` positions, its own included;
+// window < 0: the positions of its own chunk, chunks of -window positions counted from position 0; 0: all of them.
+// It never falls when pos grows.
+__host__ __device__ __forceinline__ int first_seen(int pos, int window) {
+    if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
+    return window < 0 ? pos - pos % -window : 0;
+}
+
 // Where a multi-token step finds the keys and values of positions that earlier steps stored: the paged cache line
 // ([pages, kv heads, JANIS_PAGE, head size]; position p of a sequence in page table[slot][p / JANIS_PAGE], or at
 // p % ring_len for a windowed line).  seq_start == nullptr: every sequence of the step starts at position 0 and

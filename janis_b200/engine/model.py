@@ -5,7 +5,9 @@ and an output head.  The schedule is data: a list of `LayerCall(layer,
 cache_line, write)`.  It may name a layer twice (a looped layer, each visit with
 a cache line of its own or a shared one) and may let a layer read the cache line
 that another entry writes (`write=False`: the layer projects queries only).
-Every cache line is written by exactly one entry, which comes before its readers.
+Every cache line is written by exactly one entry, which comes before its readers.  `add_embedding` adds the embedding's
+output (the stream as it was before the first entry) to the stream before the entry's first norm: what a loop does
+when it starts over.
 
 The reference runs its blocks in list order with one cache per block
 (`gemma/gemma.go:204-206`); its looped decoder visits layers repeatedly
@@ -21,6 +23,7 @@ from typing import Sequence
 import torch
 
 from ..parts.base import Block, Norm, Part, Runtime, StepContext
+from ..parts.norm import StreamPlus
 from ..weights.loader import TensorSpec
 
 
@@ -29,6 +32,7 @@ class LayerCall:
     layer: int
     cache_line: int
     write: bool = True
+    add_embedding: bool = False
 
 
 def _walk(part: Part):
@@ -85,6 +89,9 @@ class DecoderModel:
                 raise ValueError(f"cache line {line} is never written")
         self.n_cache_lines = n_lines
         self._writer = writer
+        if any(c.add_embedding for c in self.schedule):
+            if self.schedule[0].add_embedding or self.stream_width != self.hidden:
+                raise ValueError("the embedding's output joins a stream of its own width, after the first schedule entry")
 
     # -- tensors -------------------------------------------------------------
     def parts(self):
@@ -126,10 +133,15 @@ class DecoderModel:
         """Run the schedule over the step's tokens; returns the residual stream [T, hidden] float32."""
         h = ctx.ws.buf("stream.h", (ctx.n_tok, self.stream_width), torch.float32)
         self.embedding.forward(ctx.tokens, ctx, h)
+        x0 = None
+        if any(c.add_embedding for c in self.schedule):
+            x0 = self.embedding.forward(ctx.tokens, ctx, ctx.ws.buf("stream.x0", (ctx.n_tok, self.hidden), torch.float32))
         y = None
         for idx, call in enumerate(self.schedule):
             blk = self.blocks[call.layer]
             nxt = self.blocks[self.schedule[idx + 1].layer].first_norm if idx + 1 < len(self.schedule) else None
+            if idx + 1 < len(self.schedule) and self.schedule[idx + 1].add_embedding:
+                nxt = StreamPlus(nxt, x0)
             line = cache.line(call.cache_line, call.write, has_readers=call.write and self.readers[call.cache_line] > 0)
             h, y = blk.forward(h, ctx, line, y_in=y, next_norm=nxt)
         for late in ctx.shared.pop("after_step", ()):    # what parts put off until every layer has run

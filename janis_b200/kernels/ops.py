@@ -139,7 +139,7 @@ def mixers():
         _need_cuda()
         lib = build.mixers_library()
         P, I, F = c_void_p, c_int, c_float
-        lib.janis_qkv_rotate_store.argtypes = [P, I, I, P, P, P, P, I, P, I, I, I, I, I, I, P, P, P, I, P, F, I, F, P, P]
+        lib.janis_qkv_rotate_store.argtypes = [P, I, I, P, P, P, P, I, P, I, I, I, I, I, I, P, P, P, I, P, F, I, F, P, P, P, F, P]
         lib.janis_talk_attention.argtypes = [P, I, I, P, P, P, P, P, P, I, P, P, P, I, I, I, I, I, F, I, I, I, I, I, P, c_longlong, I, F, P, I, I, P, c_longlong, I, P]
         lib.janis_talk_attention_set_kernel.argtypes = [I]
         lib.janis_talk_attention_set_kernel.restype = None
@@ -170,8 +170,11 @@ def mixers():
         lib.janis_gated_recurrence_scan.argtypes = [P, I, P, c_longlong, c_longlong, P, P, P, P, I, I, P, P, P, P, P, I, P, P, I, I, F, I, I, P]
         lib.janis_gated_recurrence_rows.argtypes = [P, I, P, P, P, P, P, I, I, P, P, P, I, P, P, I, I, F, I, I, P]
         lib.janis_moe_relu2.argtypes = [P, I, P, I, I, I, I, I, I, P]
-        lib.janis_moe_route.argtypes = [P, P, I, I, I, I, I, F, I, P, I, I, I, P]
-        lib.janis_moe_expert_act.argtypes = [P, I, P, I, I, F, I, F, F, P, I, I, F, P]
+        lib.janis_moe_route.argtypes = [P, P, I, I, I, I, I, F, I, P, I, I, I, I, P]
+        lib.janis_moe_expert_act.argtypes = [P, I, P, I, I, F, I, F, F, P, I, I, F, I, P]
+        lib.janis_stream_norm.argtypes = [P, P, P, I, P, P, F, F, P, P, P, F, I, P, I, P, I, I, P]
+        lib.janis_delta_scan.argtypes = [P, I, I, I, I, P, I, I, I, I, P, P, F, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P]
+        lib.janis_delta_step.argtypes = [P, I, I, I, I, P, I, I, I, I, I, P, P, F, P, F, P, P, P, P, I, I, I, I, I, P]
         lib.janis_moe_identity_add.argtypes = [P, P, I, P, I, I, I, I, P]
         lib.janis_hc_spread.argtypes = [P, P, I, I, I, P]
         lib.janis_hc_read_norm.argtypes = [P, P, P, P, F, P, I, I, I, I, P]
@@ -703,7 +706,8 @@ def attn_prefill_rows(rows, seq_first_row, seq_len, out, H: int, G: int, hd: int
                       sinks=None, scratch=None, host_lens=None, seq_start=None, seq_slot=None, kpool=None, vpool=None,
                       page_table=None):
     """`attn_prefill` (bfloat16, tensor cores) over rows that hold q (H heads), k and v (G heads each) first and anything
-    behind them; sinks [H] float32: exp of head h's number joins its denominator.  The line of a step that continues
+    behind them; sinks [H] float32: exp of head h's number joins its denominator.  window < 0: keys are seen
+    inside the query's own chunk of -window positions, counted from the sequence's first.  The line of a step that continues
     sequences keeps every position (no ring); whether the step's own keys are stored already does not matter."""
     T, width = rows.shape
     _t(rows, "rows", torch.bfloat16, (T, None))
@@ -739,7 +743,7 @@ def attn_prefill_rows(rows, seq_first_row, seq_len, out, H: int, G: int, hd: int
 def attn_decode_rows(rows, kpool, vpool, page_table, seq_slot, seq_len, scratch, out, H: int, G: int, hd: int, scale: float,
                      window: int, chunk: int, max_chunks: int, cap: float = 0.0, sinks=None):
     """`attn_decode` (bfloat16) for rows that hold the queries first and anything behind them, over a line that keeps every
-    position; sinks as in `attn_prefill_rows`."""
+    position; sinks and window (negative: a chunk) as in `attn_prefill_rows`."""
     n_seq, width = rows.shape
     _t(rows, "rows", torch.bfloat16, (n_seq, None))
     if width < H * hd or width % 8:
@@ -875,13 +879,15 @@ def attn_decode(qkv, kpool, vpool, page_table, seq_slot, seq_len, scratch, out, 
 
 def qkv_rotate_store(rows, tok_pos, tok_seq, seq_slot, inv_qk, rot: int, inv_v, H: int, G: int, d: int, dv: int,
                      kpool=None, vpool=None, page_table=None, store: bool = True, bias=None, amplitude: float = 1.0,
-                     mix: int = 0, share: float = 0.0, v_first=None):
+                     mix: int = 0, share: float = 0.0, v_first=None, q_norm=None, k_norm=None, norm_eps: float = 0.0):
     """Rotary encoding of the first `rot` features of the queries and keys of a step (pairs i, i + rot/2), rotation
     of the values over all dv features by inv_v (None: values stay as projected), and the write of keys and values
     into the paged cache line.  rows [T, H d + G d + G dv] holds q, then k, then v; with store=False the rows hold q
     alone.  kpool [pages, G, PAGE, d], vpool [pages, G, PAGE, dv].  bias (float32, one per column of q | k | v) is added
     before anything else; `amplitude` multiplies sine and cosine of the queries' and keys' turn.  mix 1: the values are
-    also left in v_first [T, G dv]; mix 2: they become (1 - share) v + share v_first before they are stored."""
+    also left in v_first [T, G dv]; mix 2: they become (1 - share) v + share v_first before they are stored.
+    q_norm, k_norm (float32 [d] each; no bias then): every head of q and k is divided by sqrt(mean(head^2) + norm_eps) and
+    multiplied by the weight before it turns."""
     T, width = rows.shape
     _t(rows, "rows", _FLOATS, (T, None))
     if bias is not None and bias.numel() < H * d + (G * (d + dv) if store else 0):
@@ -906,7 +912,9 @@ def qkv_rotate_store(rows, tok_pos, tok_seq, seq_slot, inv_qk, rot: int, inv_v, 
         inv_v.data_ptr() if inv_v is not None else None, T, H, G, d, dv, 1 if store else 0,
         kpool.data_ptr() if store else None, vpool.data_ptr() if store else None,
         page_table.data_ptr() if store else None, stride, _t(bias, "bias", torch.float32) if bias is not None else None,
-        float(amplitude), int(mix), float(share), _t(v_first, "v_first", rows.dtype, (T, G * dv)) if mix else None, _stream()))
+        float(amplitude), int(mix), float(share), _t(v_first, "v_first", rows.dtype, (T, G * dv)) if mix else None,
+        _t(q_norm, "q_norm", torch.float32, (d,)) if q_norm is not None else None,
+        _t(k_norm, "k_norm", torch.float32, (d,)) if k_norm is not None else None, float(norm_eps), _stream()))
     return rows
 
 
@@ -978,7 +986,7 @@ def talk_attention_rows(q_rows, tok_pos, tok_seq, seq_slot, kpool, vpool, page_t
     the heads' weights mixed after the softmax; values_in_keys: the values are the first dv features of the keys.
     q_rows [T, >= H d], out [T, H dv]; max_keys bounds the keys a row sees; scratch float32 of at least
     `talk_attention_rows_floats`.  keep_first (with a window): the sequence's first positions that stay seen behind the
-    window; max_keys counts them too.  Sums are float and their order depends on the row alone."""
+    window; max_keys counts them too.  window < 0: keys are seen inside the row's own chunk of -window positions.  Sums are float and their order depends on the row alone."""
     T = q_rows.shape[0]
     _t(q_rows, "q_rows", _FLOATS, (T, None))
     n_pages = kpool.shape[0]
@@ -1354,6 +1362,93 @@ def gated_recurrence_rows(u, w, bias_r, bias_i, decay, y_rows, y_off: int, y_bia
     return out
 
 
+def stream_norm(h, r=None, scale=None, more=None, w_next=None, eps_next: float = 0.0, centred: bool = False, out=None, rows=None,
+                branch_weights=None, eps: float = 0.0, share: float = 1.0):
+    """A sublayer's result into the float32 stream, in place, and the norm behind the sum, in one pass:
+    h += scale * v + more, out = norm(h) * w_next.  r: the result [R, H], v = r; or, with branch_weights (float32 [H] each), a
+    list of one or two branches, v = share * sum_i r_i / sqrt(mean(r_i^2) + eps) * weight_i.  scale float32 [H] (None: 1), more
+    float32 [R, H] (None: nothing).  centred: norm(h) = (h - mean) / sqrt(mean((h - mean)^2) + eps_next), else
+    h / sqrt(mean(h^2) + eps_next).  With r None: out = norm(h[rows]) (all rows when `rows` is None), h untouched."""
+    H = h.shape[1]
+    parts = [] if r is None else (list(r) if branch_weights is not None else [r])
+    R = parts[0].shape[0] if parts else out.shape[0]
+    if len(parts) > 2 or (branch_weights is not None and len(branch_weights) != len(parts)):
+        raise KernelError(f"stream_norm: {len(parts)} branches with {len(branch_weights or ())} weights")
+    if parts and h.shape[0] != R:
+        raise KernelError(f"stream_norm: {h.shape[0]} rows of the stream for {R} of the result")
+    if not parts and rows is None and h.shape[0] != R:
+        raise KernelError(f"stream_norm: {h.shape[0]} input rows for {R} output rows")
+    ptr = [_t(p, "r", parts[0].dtype, (R, H)) for p in parts] + [None] * (2 - len(parts))
+    bw = [_t(w, "branch weight", torch.float32, (H,)) for w in branch_weights or ()] + [None] * 2
+    if parts:
+        _t(parts[0], "r", _FLOATS)
+    lib = mixers()
+    _check(lib, lib.janis_stream_norm(
+        _t(h, "h", torch.float32, (None, H)), ptr[0], ptr[1], _DT[parts[0].dtype] if parts else 0, bw[0], bw[1], float(eps), float(share),
+        _t(scale, "scale", torch.float32, (H,)) if scale is not None else None,
+        _t(more, "more", torch.float32, (R, H)) if more is not None else None,
+        _t(w_next, "w_next", torch.float32, (H,)) if w_next is not None else None, float(eps_next), 1 if centred else 0,
+        _t(out, "out", _FLOATS, (R, H)) if out is not None else None, _DT[out.dtype] if out is not None else 0,
+        _t(rows, "rows", torch.int32, (R,)) if rows is not None else None, R, H, _stream()))
+    return out
+
+
+DELTA_COEF = 12            # floats a token and head that `delta_scan` keeps between its two kernels
+
+
+def _delta_tables(name, x, z, offs, z_offs, H, G, d, dv, decay, dt_bias, state):
+    T = x.shape[0]
+    _t(x, "x", _FLOATS, (T, None))
+    _t(z, "z", x.dtype, (T, None))
+    _t(decay, "decay", torch.float32, (H,))
+    _t(dt_bias, "dt_bias", torch.float32, (H,))
+    _t(state, "state", torch.float32, (None, H, dv, d))
+    if offs[0] + G * d > x.shape[1] or offs[1] + G * d > x.shape[1] or offs[2] + H * dv > x.shape[1] or max(z_offs) + H > z.shape[1]:
+        raise KernelError(f"{name}: a column range lies outside its rows")
+
+
+def delta_scan(x, q_off: int, k_off: int, v_off: int, z, a_off: int, b_off: int, decay, dt_bias, q_scale: float, tok_pos, tok_seq,
+               seq_slot, seq_first_row, seq_start, seq_end, state, o_out, n_seq: int, H: int, G: int, d: int, dv: int, coef,
+               form: int = 0):
+    """The gated delta rule over the tokens each sequence brings, in order.  x [T, *] holds q [G, d], k [G, d] and v [H, dv]
+    (after the convolution) at their offsets, z [T, *] the logits za [H] and zb [H]; with k and q as unit vectors per head
+    (x / sqrt(sum(x^2) + 1e-6), q also times q_scale), g = exp(decay softplus(za + dt_bias)), beta = sigmoid(zb):
+    S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  decay (negative), dt_bias float32 [H]; state float32
+    [slots, H, dv, d] (S^T) is read and written back for slots >= 0; coef float32 scratch [T, H, DELTA_COEF]; o_out float32
+    [T, H dv].  form: 1 or 2 fixes how many columns a group of lanes takes (0: chosen per launch)."""
+    T = x.shape[0]
+    _delta_tables("delta_scan", x, z, (q_off, k_off, v_off), (a_off, b_off), H, G, d, dv, decay, dt_bias, state)
+    for name, tab, n in (("tok_pos", tok_pos, T), ("tok_seq", tok_seq, T), ("seq_slot", seq_slot, n_seq),
+                         ("seq_first_row", seq_first_row, n_seq), ("seq_start", seq_start, n_seq), ("seq_end", seq_end, n_seq)):
+        _t(tab, name, torch.int32)
+        if tab.numel() < n:
+            raise KernelError(f"delta_scan: {name} shorter than the step")
+    lib = mixers()
+    _check(lib, lib.janis_delta_scan(
+        x.data_ptr(), x.shape[1], int(q_off), int(k_off), int(v_off), z.data_ptr(), z.shape[1], int(a_off), int(b_off), _DT[x.dtype],
+        decay.data_ptr(), dt_bias.data_ptr(), float(q_scale), _t(coef, "coef", torch.float32, (T, H, DELTA_COEF)), tok_pos.data_ptr(),
+        tok_seq.data_ptr(), seq_slot.data_ptr(), seq_first_row.data_ptr(), seq_start.data_ptr(), seq_end.data_ptr(), state.data_ptr(),
+        _t(o_out, "o_out", torch.float32, (T, H * dv)), n_seq, T, H, G, d, dv, int(form), _stream()), kernels=2)
+    return o_out
+
+
+def delta_step(x, q_off: int, k_off: int, v_off: int, z, a_off: int, b_off: int, g_off: int, decay, dt_bias, q_scale: float, weight,
+               eps: float, tok_seq, seq_slot, state, out, H: int, G: int, d: int, dv: int):
+    """`delta_scan` for a step whose sequences bring one token each, and what follows it: out[t, h] = o / sqrt(mean(o^2) + eps)
+    * weight * silu(gate), the gate's logits [H, dv] at g_off of z; weight float32 [dv]; out [T, H dv] of x's dtype."""
+    T = x.shape[0]
+    _delta_tables("delta_step", x, z, (q_off, k_off, v_off), (a_off, b_off), H, G, d, dv, decay, dt_bias, state)
+    if g_off + H * dv > z.shape[1] or tok_seq.numel() < T:
+        raise KernelError("delta_step: the gate lies outside its rows, or tok_seq is shorter than the step")
+    lib = mixers()
+    _check(lib, lib.janis_delta_step(
+        x.data_ptr(), x.shape[1], int(q_off), int(k_off), int(v_off), z.data_ptr(), z.shape[1], int(a_off), int(b_off), int(g_off),
+        _DT[x.dtype], decay.data_ptr(), dt_bias.data_ptr(), float(q_scale), _t(weight, "weight", torch.float32, (dv,)), float(eps),
+        _t(tok_seq, "tok_seq", torch.int32), _t(seq_slot, "seq_slot", torch.int32), state.data_ptr(),
+        _t(out, "out", x.dtype, (T, H * dv)), T, H, G, d, dv, _stream()))
+    return out
+
+
 def group_norm(h, res, alpha: float, weight, eps: float, groups: int, out, rows=None):
     """RMS norm in `groups` equal runs of the row, each divided by its own sqrt(mean(run^2) + eps), the whole times
     weight.  With res: h <- norm(alpha h + res) on the float32 stream in place, and out (when given) = h rounded.
@@ -1505,7 +1600,7 @@ def head_linear(x, x_head: int, x_off: int, w, out, o_head: int, o_off: int):
 
 
 def moe_route(z, correction, n_experts: int, group_count: int, group_keep: int, top: int, scale: float,
-              shared_gate: bool, out, n_identity: int = 0, softmax: bool = False, group_best: bool = False):
+              shared_gate: bool, out, n_identity: int = 0, softmax: bool = False, group_best: bool = False, raw: bool = False):
     """The router's weights per token and expert, 0 for experts that were not chosen: s = sigmoid(z), choice scores
     s + correction, the best group_keep of group_count groups (by the sum of a group's two largest choice scores), the
     `top` largest choice scores among their experts, w = s / (sum of the chosen s + 1e-20) * scale.  With
@@ -1513,7 +1608,7 @@ def moe_route(z, correction, n_experts: int, group_count: int, group_keep: int, 
     softmax: s = softmax(z) over all entries instead.  n_identity: that many more entries behind the experts in z and
     correction (before the gate's column); they are scored and chosen like experts, and the weights of the chosen ones
     add up in one more column at the end of out.  group_best: a group's score is its largest choice score alone.
-    correction may be None (zeros)."""
+    correction may be None (zeros).  raw: the chosen scores themselves (times scale) are the weights."""
     T = z.shape[0]
     n = n_experts + n_identity
     cols_in = n + (1 if shared_gate else 0)
@@ -1522,7 +1617,7 @@ def moe_route(z, correction, n_experts: int, group_count: int, group_keep: int, 
     _check(lib, lib.janis_moe_route(_t(z, "z", torch.float32, (T, cols_in)), _t(correction, "correction", torch.float32, (n,)) if correction is not None else None,
                                     T, n_experts, int(group_count), int(group_keep), int(top), float(scale),
                                     1 if shared_gate else 0, _t(out, "out", torch.float32, (T, cols_out)), int(n_identity),
-                                    1 if softmax else 0, 1 if group_best else 0, _stream()))
+                                    1 if softmax else 0, 1 if group_best else 0, 1 if raw else 0, _stream()))
     return out
 
 
@@ -1536,18 +1631,19 @@ def moe_identity_add(out, y, wts, col: int):
 
 
 def moe_expert_act(gu, wts, n_experts: int, ff: int, limit: float, shared_ff: int, shared_limit: float, alpha: float, out,
-                   up_add: float = 1.0):
+                   up_add: float = 1.0, weight_in: bool = False):
     """out[t, e * ff + j] = wts[t, e] * g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit,
     limit); gu [T, 2 (E ff + shared_ff)] holds each expert's ff gate columns followed by its ff up columns, the
     shared expert (weight wts[t, E], its own limit) last; out [T, E ff + shared_ff].  up_add replaces the 1 (0: the plain
-    gated form); wts may have further columns behind the ones used."""
+    gated form); wts may have further columns behind the ones used.  weight_in: the weight stands on the expert's input:
+    gate and up are multiplied by it first and the result is not."""
     T = gu.shape[0]
     total = n_experts * ff + shared_ff
     lib = mixers()
     _check(lib, lib.janis_moe_expert_act(_t(gu, "gu", _FLOATS, (T, 2 * total)), _DT[gu.dtype],
                                          _t(wts, "wts", torch.float32, (T, None)),
                                          n_experts, ff, float(limit), int(shared_ff), float(shared_limit), float(alpha),
-                                         _t(out, "out", gu.dtype, (T, total)), T, wts.shape[1], float(up_add), _stream()))
+                                         _t(out, "out", gu.dtype, (T, total)), T, wts.shape[1], float(up_add), 1 if weight_in else 0, _stream()))
     return out
 
 

@@ -27,7 +27,8 @@ sequence after sequence without padding):
   `in_weight()` [columns, hidden] and `out_weight()` [hidden, features] (and keeps
   neither), and `join(rows, col0, ctx, line, z, z0, scale)` goes from its columns
   of the shared product's rows to its features (times `scale`) in z's columns from
-  z0.  `joins`: "any", "first" (its columns must be the rows' first) or "" (it
+  z0; `finish(rows, col0, ctx, line, out)` goes from its columns to its own output (keeping `out_weight`'s matrix), for
+  mixers that share the first product alone.  `joins`: "any", "first" (its columns must be the rows' first) or "" (it
   cannot).
 * `FeedForward.forward(x, ctx)` -> [T, hidden].
 * `Block.forward(h, ctx, line, y_in=None, next_norm=None)` -> (h, y_next): h is the
@@ -226,6 +227,9 @@ class Mixer(Part):
         raise NotImplementedError(f"{type(self).__name__} shares its products with no other mixer")
 
     def join(self, rows, col0: int, ctx: StepContext, line, z, z0: int, scale: float) -> None:
+        raise NotImplementedError(f"{type(self).__name__} shares its products with no other mixer")
+
+    def finish(self, rows, col0: int, ctx: StepContext, line, out):
         raise NotImplementedError(f"{type(self).__name__} shares its products with no other mixer")
 
 

@@ -7,7 +7,8 @@ out = h + N_post_ff(r).  Without a feed-forward (`feed_forward=None`) a layer is
 
 `PreNormBlock` is the usual arrangement without the norms after the sublayers
 (`qwen/block.go:58-61`): h = x + Mixer(N_in(x)); out = h + FF(N_pre_ff(h)); without a feed-forward the first
-line alone.
+line alone.  With `mixer_scale_name` and `ff_scale_name` a stored factor per feature multiplies each sublayer's result before
+the sum.
 
 `PostNormBlock` norms after the sum, and the stream that goes on is the normed one: x <- N1(a x + Mixer(x));
 x <- N2(a x + FF(x)) with a constant a; the sublayers read the stream itself (rounded to the activation type).
@@ -21,7 +22,7 @@ norm to its own result, which saves a pass over the stream per layer.
 from __future__ import annotations
 
 from .base import Block, FeedForward, Mixer, Norm, StepContext
-from .norm import plain_residual_add
+from .norm import FeatureScale, plain_residual_add
 
 import torch
 
@@ -57,17 +58,23 @@ class SandwichBlock(Block):
 
 
 class PreNormBlock(Block):
-    def __init__(self, mixer: Mixer, feed_forward: FeedForward | None, input_norm: Norm, pre_ff_norm: Norm | None = None):
+    def __init__(self, mixer: Mixer, feed_forward: FeedForward | None, input_norm: Norm, pre_ff_norm: Norm | None = None,
+                 width: int = 0, mixer_scale_name: str | None = None, ff_scale_name: str | None = None):
         if feed_forward is not None and pre_ff_norm is None:
             raise ValueError("a block with a feed-forward needs the norm before it")
+        if (mixer_scale_name or ff_scale_name) and width < 1:
+            raise ValueError("factors on a sublayer's result need the model's width")
+        self.mixer_scale = FeatureScale(width, mixer_scale_name) if mixer_scale_name else None
+        self.ff_scale = FeatureScale(width, ff_scale_name) if ff_scale_name else None
         self.mixer, self.feed_forward = mixer, feed_forward
         self.first_norm = input_norm
         self.pre_ff_norm = pre_ff_norm
 
     def sub_parts(self):
+        scales = [s for s in (self.mixer_scale, self.ff_scale) if s is not None]
         if self.feed_forward is None:
-            return [self.first_norm, self.mixer]
-        return [self.first_norm, self.mixer, self.pre_ff_norm, self.feed_forward]
+            return [self.first_norm, self.mixer, *scales]
+        return [self.first_norm, self.mixer, self.pre_ff_norm, self.feed_forward, *scales]
 
     def forward(self, h, ctx: StepContext, line, y_in=None, next_norm: Norm | None = None):
         T, H = h.shape
@@ -76,11 +83,11 @@ class PreNormBlock(Block):
         r = self.mixer.forward(y, ctx, line)
         if self.feed_forward is None:
             return h, plain_residual_add(h, r, ctx, next_norm,
-                                         ctx.ws.buf("block.y", (T, H), dt) if next_norm is not None else None)
-        y = plain_residual_add(h, r, ctx, self.pre_ff_norm, ctx.ws.buf("block.y", (T, H), dt))
+                                         ctx.ws.buf("block.y", (T, H), dt) if next_norm is not None else None, self.mixer_scale)
+        y = plain_residual_add(h, r, ctx, self.pre_ff_norm, ctx.ws.buf("block.y", (T, H), dt), self.mixer_scale)
         r = self.feed_forward.forward(y, ctx)
         y_next = plain_residual_add(h, r, ctx, next_norm,
-                                    ctx.ws.buf("block.y", (T, H), dt) if next_norm is not None else None)
+                                    ctx.ws.buf("block.y", (T, H), dt) if next_norm is not None else None, self.ff_scale)
         return h, y_next
 
 

@@ -17,7 +17,9 @@ Expert (no biases):  g = min(W_gate y, limit),  u = clamp(W_up y, -limit, limit)
 Other forms of the same parts: `score="softmax"` takes s = softmax(W_r y) over all router entries instead of the
 logistic function; `act="silu"` is the plain gated expert W_down (silu(W_gate y) * (W_up y)) without limits; and
 `n_identity` router entries behind the experts have no tensors and return their input, so that a token's chosen
-identity entries add (sum of their w) y to the output.  `act="relu2"` is the plain expert W_down relu(W_up y)^2 (no gate
+identity entries add (sum of their w) y to the output.  `renormalize=False`: w_e = s_e * scale, the chosen scores as they
+are.  `weight_on="input"`: a weight multiplies its expert's input instead of its output, sum over chosen expert_e(w_e y);
+gate and up are linear in the input, so the activation kernel multiplies both by w_e.  `act="relu2"` is the plain expert W_down relu(W_up y)^2 (no gate
 matrices).  Without names["correction"] the scores choose; `group_score="best"`: a group's score is its largest c alone.
 Without names["shared_gate"] the shared expert is added as it is (plain experts only).
 
@@ -42,7 +44,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden: int, n_experts: int, top: int, expert_ff: int, limit: float, scale: float,
                  names: dict[str, str], group_count: int = 1, group_keep: int = 1, shared_ff: int = 0,
                  shared_limit: float = 0.0, gate_alpha: float = 1.702, init_std: float = 0.02, score: str = "sigmoid",
-                 act: str = "clamped_swish", n_identity: int = 0, group_score: str = "best_two"):
+                 act: str = "clamped_swish", n_identity: int = 0, group_score: str = "best_two", renormalize: bool = True,
+                 weight_on: str = "output"):
         """names: "router", "correction" (optional), "expert" (a pattern with {e} and {w}: w is gate, up or down), and with a
         shared expert "shared" (a pattern with {w}) and "shared_gate" (optional with act="relu2")."""
         for k in ("router", "expert") + (("shared",) if shared_ff else ()) + (("shared_gate",) if shared_ff and act != "relu2" else ()):
@@ -54,6 +57,9 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"unknown expert activation {act!r} (known: clamped_swish, relu2, silu)")
         if group_score not in ("best_two", "best"):
             raise ValueError(f"unknown group score {group_score!r} (known: best, best_two)")
+        if weight_on not in ("output", "input") or (weight_on == "input" and (act == "relu2" or shared_ff)):
+            raise ValueError(f"weights stand on the output, or on the input of gated experts without a shared one, found {weight_on!r}")
+        self.renormalize, self.weight_on = bool(renormalize), weight_on
         self.group_score = group_score
         self.mats = ("up", "down") if act == "relu2" else ("gate", "up", "down")
         self.score, self.act, self.n_identity = score, act, int(n_identity or 0)
@@ -138,7 +144,7 @@ class RoutedExperts(FeedForward):
         ops.moe_route(z, self.correction, E, self.group_count, self.group_keep, self.top, self.scale,
                       self.gated_shared, wts,
                       **({} if plain else {"n_identity": self.n_identity, "softmax": self.score == "softmax"}),
-                      **({"group_best": True} if self.group_score == "best" else {}))
+                      **({"group_best": True} if self.group_score == "best" else {}), **({} if self.renormalize else {"raw": True}))
         out = ws.buf("ffn.out", (T, self.hidden), rt.dtype)
         if self.total_ff and self.act == "relu2":
             a = rt.linear(x, self.w_gu, ws.buf("moe.act", (T, self.total_ff), rt.dtype))
@@ -148,7 +154,8 @@ class RoutedExperts(FeedForward):
             gu = rt.linear(x, self.w_gu, ws.buf("moe.gu", (T, 2 * self.total_ff), rt.dtype))
             a = ws.buf("moe.act", (T, self.total_ff), rt.dtype)
             ops.moe_expert_act(gu, wts, E, self.expert_ff, self.limit, self.shared_ff, self.shared_limit, self.gate_alpha, a,
-                               **({} if plain else {"up_add": 0.0 if self.act == "silu" else 1.0}))
+                               **({} if plain else {"up_add": 0.0 if self.act == "silu" else 1.0}),
+                               **({"weight_in": True} if self.weight_on == "input" else {}))
             rt.linear(a, self.w_down, out)
         else:
             out.zero_()

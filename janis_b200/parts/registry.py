@@ -40,6 +40,7 @@ def make(family: str, kind: str, **params):
 def _register_builtin() -> None:
     from .attention import SoftmaxAttention
     from .block import PostNormBlock, PreNormBlock, SandwichBlock
+    from .delta_rule import GatedDeltaRule
     from .embedding import Embedding, LMHead
     from .feedforward import DenseMLP, GatedMLP
     from .filtered_attention import FilteredAttention
@@ -50,7 +51,7 @@ def _register_builtin() -> None:
     from .linear_attention import GatedLinearAttention
     from .talking_attention import TalkingHeadsAttention
     from .moe import RoutedExperts
-    from .norm import DynamicTanh, GroupRMSNorm, RMSNorm
+    from .norm import DynamicTanh, GroupRMSNorm, LayerNorm, RMSNorm
     from .parallel import ParallelMixers
     from .state_space import DualityMixer, SelectiveScanMixer
     from .position import NoPosition, RotaryEncoding
@@ -61,6 +62,7 @@ def _register_builtin() -> None:
     register("mixer", "latent_attention", LatentAttention)                 # one compressed row cached per position, a sink per head, a window
     register("mixer", "gated_linear_attention", GatedLinearAttention)     # a matrix of state per head, decays per key channel
     register("mixer", "matrix_memory", MatrixMemory)                      # a matrix, a normaliser and a running maximum per head, exponential gates
+    register("mixer", "gated_delta_rule", GatedDeltaRule)                 # a matrix of state per head, corrected towards each value
     register("mixer", "selective_scan", SelectiveScanMixer)               # a state per channel, step sizes through a low rank
     register("mixer", "state_space_duality", DualityMixer)                # a scalar decay per head, grouped B and C
     register("mixer", "gated_recurrence", GatedRecurrenceMixer)           # a number of state per channel, decays gated by the input
@@ -69,6 +71,7 @@ def _register_builtin() -> None:
     register("feed_forward", "dense_mlp", DenseMLP)                       # up, activation, down, with biases
     register("feed_forward", "routed_experts", RoutedExperts)             # a router over small gated experts, a shared one
     register("norm", "rms_norm", RMSNorm)
+    register("norm", "layer_norm", LayerNorm)
     register("norm", "dynamic_tanh", DynamicTanh)
     register("norm", "group_rms_norm", GroupRMSNorm)       # each run of the row by its own root mean square; norms the stream in place
     register("norm", "hyper_read", HyperRead)              # a weighted sum of the stream's copies, then the RMS norm

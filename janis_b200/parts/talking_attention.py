@@ -29,7 +29,11 @@ per head): exp(sink_h) joins the denominator instead of 1.  The position encodin
 (1 - m) v + m v_first with the stored number m (names["vmix"]) before they are cached, v_first being the values of the
 same token in the layer that left them.
 
-In the serving dtype an attention without head mixing, blocks, turned values or kept positions, with values as wide as
+`head_norm_eps` with names["q_norm"] and names["k_norm"]: every head of q and k is divided by sqrt(mean(head^2) + eps) and
+multiplied by a stored weight of d features (one for all heads of q, one for those of k) before it turns.  `cap`: a scaled
+score s becomes cap tanh(s / cap) before anything else.
+
+In the serving dtype an attention without head mixing, turned values or kept positions, with values as wide as
 its keys, runs the kernels of `SoftmaxAttention` (a prompt step reads its own keys and values from the projected rows).
 
 Keys and values live in a paged cache line with separate head sizes.  A step writes its keys and values first
@@ -53,7 +57,7 @@ class TalkingHeadsAttention(Mixer):
                  position: RotaryEncoding, names: dict[str, str], value_position: RotaryEncoding | None = None,
                  block: int = 0, sink: bool = False, own_kv: bool = True, init_std: float = 0.02, window: int = 0,
                  keep_first: int = 0, values_from_keys: bool = False, unit_norm_eps: float | None = None,
-                 gate: str = "element", value_mix: str | None = None):
+                 gate: str = "element", value_mix: str | None = None, cap: float = 0.0, head_norm_eps: float | None = None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads do not divide over {n_kv_heads} key/value heads")
         if gate not in ("head", "element"):
@@ -74,6 +78,12 @@ class TalkingHeadsAttention(Mixer):
         if (biases or value_mix) and (not own_kv or values_from_keys or value_position is not None):
             raise ValueError("biases and mixed values belong to a layer with plain values of its own")
         self.value_mix, self.biased = value_mix, bool(biases)
+        if (head_norm_eps is not None) != ("q_norm" in names) or ("q_norm" in names) != ("k_norm" in names):
+            raise ValueError("normed heads need head_norm_eps and the checkpoint names of both weights, 'q_norm' and 'k_norm'")
+        if head_norm_eps is not None and (biases or not own_kv or values_from_keys):
+            raise ValueError("normed heads belong to a layer with keys and values of its own and without biases")
+        self.head_norm_eps = None if head_norm_eps is None else float(head_norm_eps)
+        self.cap = float(cap or 0.0)
         need = (("q", "k", "o") if values_from_keys else ("q", "k", "v", "o")) if own_kv else ("q", "o")
         for k in need:
             if k not in names:
@@ -92,7 +102,7 @@ class TalkingHeadsAttention(Mixer):
         self.position, self.value_position = position, value_position
         self.names = dict(names)
         self.init_std = init_std
-        self.w_qkv = self.w_o = self.talk = self.bias = self.sink_values = None
+        self.w_qkv = self.w_o = self.talk = self.bias = self.sink_values = self.wq_norm = self.wk_norm = None
         self.mix_share = 0.0
 
     def tensor_specs(self):
@@ -109,6 +119,8 @@ class TalkingHeadsAttention(Mixer):
         if self.biased:
             specs.update({n["q_bias"]: TensorSpec((H * d,), init_std=s), n["k_bias"]: TensorSpec((G * d,), init_std=s),
                           n["v_bias"]: TensorSpec((G * dv,), init_std=s)})
+        if self.head_norm_eps is not None:
+            specs.update({n[k]: TensorSpec((d,), init_std=0.1, init_mean=1.0) for k in ("q_norm", "k_norm")})
         if "sink" in n:
             specs[n["sink"]] = TensorSpec((H,), init_std=1.0)
         if self.value_mix == "mix":
@@ -154,6 +166,8 @@ class TalkingHeadsAttention(Mixer):
         f32 = lambda k: store.get(n[k]).to(torch.float32)
         self.bias = torch.cat([f32("q_bias"), f32("k_bias"), f32("v_bias")]).contiguous() if self.biased else None
         self.sink_values = f32("sink").contiguous() if "sink" in n else None
+        if self.head_norm_eps is not None:
+            self.wq_norm, self.wk_norm = f32("q_norm").contiguous(), f32("k_norm").contiguous()
         self.mix_share = float(f32("vmix").reshape(()).item()) if self.value_mix == "mix" else 0.0
         self.talk = store.get(n["talk"]).to(torch.float32).contiguous() if "talk" in n else None
 
@@ -177,14 +191,19 @@ class TalkingHeadsAttention(Mixer):
         return self.value_dim if self.gate == "head" else 1
 
     def forward(self, x, ctx: StepContext, line):
-        rt, ws, ops = ctx.rt, ctx.ws, ctx.rt.ops
+        rt, ws = ctx.rt, ctx.ws
         T = ctx.n_tok
         rows = ws.buf("tattn.rows", (T, self.w_qkv.shape[0]), rt.dtype)      # (the product's columns: the gate's, and padding, last)
         rt.linear(x, self.w_qkv, rows)
+        return self.finish(rows, 0, ctx, line, ws.buf("mixer.out", (T, self.hidden), rt.dtype))
+
+    def finish(self, rows, col0: int, ctx: StepContext, line, out):
+        if col0:
+            raise ValueError("an attention's columns are the first of the rows it shares")
         att = self._attend(rows, ctx, line)
         if "g" in self.names:
-            ops.sigmoid_gate(att, rows, self._gate_off(), per=self._gate_run())
-        return rt.linear(att, self.w_o, ws.buf("mixer.out", (T, self.hidden), rt.dtype))
+            ctx.rt.ops.sigmoid_gate(att, rows, self._gate_off(), per=self._gate_run())
+        return ctx.rt.linear(att, self.w_o, out)
 
     def join(self, rows, col0: int, ctx: StepContext, line, z, z0: int, scale: float) -> None:
         if col0:
@@ -202,7 +221,7 @@ class TalkingHeadsAttention(Mixer):
         inv_v = self.value_position.inv_freq if self.value_position is not None else None
         neighbours = self.position.pairs == "neighbours" and self.position.rot > 0
         if self.values_from_keys or self.unit_norm_eps is not None or neighbours:
-            if inv_v is not None or not self.own_kv or self.position.amplitude != 1.0 or self.biased or self.value_mix:
+            if inv_v is not None or not self.own_kv or self.position.amplitude != 1.0 or self.biased or self.value_mix or self.head_norm_eps is not None:
                 raise NotImplementedError("turned or mixed values, biases, a borrowed line or an amplitude together with normed or neighbouring pairs")
             if not self.values_from_keys:
                 raise NotImplementedError("normed or neighbouring pairs beside a value projection of its own")
@@ -220,6 +239,8 @@ class TalkingHeadsAttention(Mixer):
                 ctx.shared["first values"] = extras["v_first"]
             elif self.value_mix == "mix":
                 extras.update(mix=2, share=self.mix_share, v_first=ctx.shared["first values"])
+            if self.head_norm_eps is not None:
+                extras.update(q_norm=self.wq_norm, k_norm=self.wk_norm, norm_eps=self.head_norm_eps)
             ops.qkv_rotate_store(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, self.position.inv_freq, self.position.rot,
                                  inv_v, H, G, d, dv, kv.k if self.own_kv else None, kv.v if self.own_kv else None,
                                  kv.table if self.own_kv else None, store=self.own_kv, **extras)
@@ -231,19 +252,21 @@ class TalkingHeadsAttention(Mixer):
             more["keep_first"] = self.keep_first
         if self.sink_values is not None:
             more["sink_values"] = self.sink_values
+        if self.cap:
+            more["cap"] = self.cap
         decode = ctx.mode == "decode"
         max_keys, n_chunks, scratch = 0, 1, None
         rows_floats = 0
-        if (decode and rt.dtype == torch.bfloat16 and not self.block and self.talk is None and inv_v is None
+        if (decode and rt.dtype == torch.bfloat16 and not (self.block and self.window) and self.talk is None and inv_v is None
                 and (not self.sink or self.sink_values is not None) and hasattr(ops, "talk_attention_rows_floats")):
             # a decode step in the serving dtype with nothing the kernels that take single rows leave out: keys and
             # values read once, 16 bytes a lane
-            max_keys = min(ctx.len_bound, self.window + self.keep_first) if self.window else ctx.len_bound
+            max_keys = min(ctx.len_bound, (self.window or self.block) + self.keep_first) if self.window or self.block else ctx.len_bound
             rows_floats = ops.talk_attention_rows_floats(rt.dtype, T, H, G, d, dv, max_keys)
         if rows_floats:
             return ops.talk_attention_rows(rows, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, kv.k, kv.v, kv.table, None, att, H, G, d, dv,
                                            self.scale, ws.buf("tattn.rows_scratch", (rows_floats,), torch.float32), max_keys,
-                                           sink=self.sink, window=self.window, **more)
+                                           sink=self.sink, window=self.window or -self.block, **more)
         if decode:
             # a decode row's keys over several CTAs when the rows alone would leave most of the GPU idle: about a
             # CTA an SM in all, none with fewer than 128 keys (the bound on the lengths is the host's)
@@ -259,20 +282,21 @@ class TalkingHeadsAttention(Mixer):
 
     def _plain_heads(self, rt) -> bool:
         """Whether the kernels of whole heads (one head a CTA, keys and values of one size) take this attention."""
-        return (self.talk is None and not self.block and self.value_position is None and not self.keep_first and self.own_kv
+        return (self.talk is None and not (self.block and self.window) and self.value_position is None and not self.keep_first and self.own_kv
                 and not self.values_from_keys and (not self.sink or self.sink_values is not None) and hasattr(rt.ops, "attn_rows_sizes")
                 and rt.ops.attn_rows_sizes(rt.dtype, self.n_heads, self.n_kv_heads, self.key_dim, self.value_dim))
 
     def _attend_plain(self, rows, ctx: StepContext, kv, att):
         rt, ws, ops = ctx.rt, ctx.ws, ctx.rt.ops
         H, G, d = self.n_heads, self.n_kv_heads, self.key_dim
+        seen = self.window or -self.block                      # (a negative window: chunks of that many positions)
         if ctx.mode == "decode":
-            chunk, max_chunks = decode_geometry(ctx, rt.sm_count, d, G, self.window)
+            chunk, max_chunks = decode_geometry(ctx, rt.sm_count, d, G, abs(seen))
             scratch = ws.buf("attn.partial", (ops.attn_decode_scratch_floats(ctx.n_seq, H, d, max_chunks),), torch.float32)
             return ops.attn_decode_rows(rows, kv.k, kv.v, kv.table, ctx.seq_slot, ctx.seq_end, scratch, att, H, G, d, self.scale,
-                                        self.window, chunk, max_chunks, sinks=self.sink_values)
+                                        seen, chunk, max_chunks, cap=self.cap, sinks=self.sink_values)
         n_scratch = ops.attn_prefill_scratch_floats(ctx.n_tok, ctx.n_seq, H, d, rt.dtype)
         scratch = ws.buf("attn.prefill_partial", (n_scratch,), torch.float32) if n_scratch else None
         before = dict(seq_start=ctx.seq_start, seq_slot=ctx.seq_slot, kpool=kv.k, vpool=kv.v, page_table=kv.table) if ctx.extends else {}
-        return ops.attn_prefill_rows(rows, ctx.seq_first_row, ctx.seq_end, att, H, G, d, self.scale, self.window,
+        return ops.attn_prefill_rows(rows, ctx.seq_first_row, ctx.seq_end, att, H, G, d, self.scale, seen, cap=self.cap,
                                      sinks=self.sink_values, scratch=scratch, host_lens=ctx.step_lens, **before)

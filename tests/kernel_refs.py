@@ -344,7 +344,8 @@ def _turn(x, pos, inv, sign=1.0):
 
 
 def qkv_rotate_store(rows, tok_pos, tok_seq, seq_slot, inv_qk, rot, inv_v, H, G, d, dv, kpool=None, vpool=None,
-                     page_table=None, store=True, bias=None, amplitude=1.0, mix=0, share=0.0, v_first=None):
+                     page_table=None, store=True, bias=None, amplitude=1.0, mix=0, share=0.0, v_first=None, q_norm=None, k_norm=None,
+                     norm_eps=0.0):
     T = rows.shape[0]
     for t in range(T):
         pos = int(tok_pos[t])
@@ -353,6 +354,9 @@ def qkv_rotate_store(rows, tok_pos, tok_seq, seq_slot, inv_qk, rot, inv_v, H, G,
         x = qk.double()
         if bias is not None:
             x = x + bias[:n * d].double().view(n, d)
+        if q_norm is not None:
+            x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + norm_eps)
+            x = torch.cat([x[:H] * q_norm.double(), x[H:] * k_norm.double()])
         y = _turn(x, pos, inv_qk)
         y[:, :2 * inv_qk.numel()] *= float(np.float32(amplitude))
         qk.copy_(y.to(rows.dtype))
@@ -388,6 +392,8 @@ def talk_attention(q_rows, tok_pos, tok_seq, seq_slot, kpool, vpool, page_table,
             out[t] = 0
             continue
         first = (pos // block) * block if block > 0 else 0
+        if window < 0:                         # a chunk of -window positions
+            first = pos - pos % -window
         if window > 0:
             first = max(first, pos - window + 1)
         js = list(range(min(keep_first, first) if window > 0 else 0)) + list(range(first, pos + 1))
@@ -670,7 +676,7 @@ def head_linear(x, x_head, x_off, w, out, o_head, o_off):
 
 
 def moe_route(z, correction, n_experts, group_count, group_keep, top, scale, shared_gate, out, n_identity=0, softmax=False,
-              group_best=False):
+              group_best=False, raw=False):
     T = z.shape[0]
     real = n_experts
     n_experts = real + n_identity          # the entries that are scored and chosen
@@ -683,7 +689,7 @@ def moe_route(z, correction, n_experts, group_count, group_keep, top, scale, sha
         kept = sorted(range(group_count), key=lambda g: (-gs[g], g))[:group_keep]
         cand = [e for g in sorted(kept) for e in range(g * per, (g + 1) * per)]
         chosen = sorted(cand, key=lambda e: (-float(c[t, e]), e))[:top]
-        total = sum(float(s[t, e]) for e in chosen) + 1e-20
+        total = 1.0 if raw else sum(float(s[t, e]) for e in chosen) + 1e-20
         for e in chosen:
             if e < real:
                 out[t, e] = float(s[t, e]) / total * scale
@@ -699,11 +705,14 @@ def moe_identity_add(out, y, wts, col):
     return out
 
 
-def moe_expert_act(gu, wts, n_experts, ff, limit, shared_ff, shared_limit, alpha, out, up_add=1.0):
+def moe_expert_act(gu, wts, n_experts, ff, limit, shared_ff, shared_limit, alpha, out, up_add=1.0, weight_in=False):
     T = gu.shape[0]
     v = gu.double()
     E = n_experts
     g = v[:, :2 * E * ff].view(T, E, 2, ff)
+    if weight_in:                              # the weight on the expert's input: gate and up are linear in it
+        g = g * wts[:, :E].double()[:, :, None, None]
+        wts = torch.ones_like(wts)
     gate, up = torch.clamp(g[:, :, 0], max=limit), torch.clamp(g[:, :, 1], min=-limit, max=limit)
     a = gate * torch.sigmoid(alpha * gate) * (up + up_add) * wts[:, :E].double()[:, :, None]
     out[:, :E * ff] = a.reshape(T, E * ff).to(out.dtype)
@@ -867,3 +876,77 @@ def gated_recurrence_rows(u, w, bias_r, bias_i, decay, y_rows, y_off, y_bias, to
     slots = torch.tensor([int(seq_slot[int(tok_seq[t])]) for t in range(T)], dtype=torch.int32)
     return gated_recurrence_scan(u, gates, block, bias_r, bias_i, decay, y_rows, y_off, y_bias, slots, rows,
                                  torch.zeros_like(rows), torch.ones_like(rows), T, state, out, o_off, scale)
+
+
+# ---------------------------------------------------------------------------
+# a sublayer's result into the stream with the norm behind it; the gated delta rule
+# ---------------------------------------------------------------------------
+
+def stream_norm(h, r=None, scale=None, more=None, w_next=None, eps_next=0.0, centred=False, out=None, rows=None,
+                branch_weights=None, eps=0.0, share=1.0):
+    x = h.double()
+    if r is not None:
+        if branch_weights is not None:
+            v = sum(share * b.double() / torch.sqrt((b.double() ** 2).mean(-1, keepdim=True) + eps) * w.double()
+                    for b, w in zip(r, branch_weights))
+        else:
+            v = r.double()
+        x = x + (v * scale.double() if scale is not None else v)
+        if more is not None:
+            x = x + more.double()
+        h.copy_(x.float())
+        x = h.double()
+    elif rows is not None:
+        x = x[rows.long()]
+    if w_next is not None:
+        c = x - x.mean(-1, keepdim=True) if centred else x
+        out.copy_((c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps_next) * w_next.double()).to(out.dtype))
+    return out
+
+
+DELTA_COEF = 12
+
+
+def _delta_token(S, x, q_off, k_off, v_off, zrow, a_off, b_off, decay, dt_bias, q_scale, H, G, d, dv):
+    """One token of the gated delta rule on S [H, dv, d] (float64, in place); returns o [H, dv]."""
+    rep = H // G
+
+    def unit(off):
+        v = x[off:off + G * d].double().view(G, d)
+        return (v / torch.sqrt((v * v).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(rep, dim=0)
+
+    q, k, v = unit(q_off) * q_scale, unit(k_off), x[v_off:v_off + H * dv].double().view(H, dv)
+    za = zrow[a_off:a_off + H].double() + dt_bias.double()
+    g = torch.exp(decay.double() * torch.logaddexp(za, torch.zeros_like(za)))
+    beta = torch.sigmoid(zrow[b_off:b_off + H].double())
+    S *= g[:, None, None]
+    u = beta[:, None] * (v - torch.einsum("hvd,hd->hv", S, k))
+    S += u[:, :, None] * k[:, None, :]
+    return torch.einsum("hvd,hd->hv", S, q)
+
+
+def delta_scan(x, q_off, k_off, v_off, z, a_off, b_off, decay, dt_bias, q_scale, tok_pos, tok_seq, seq_slot, seq_first_row,
+               seq_start, seq_end, state, o_out, n_seq, H, G, d, dv, coef=None, form=0):
+    for s in range(n_seq):
+        slot, row0, n = int(seq_slot[s]), int(seq_first_row[s]), int(seq_end[s]) - int(seq_start[s])
+        S = state[slot].double() if slot >= 0 else torch.zeros(H, dv, d, dtype=torch.float64)
+        for t in range(row0, row0 + n):
+            o_out[t] = _delta_token(S, x[t], q_off, k_off, v_off, z[t], a_off, b_off, decay, dt_bias, q_scale, H, G, d,
+                                    dv).reshape(-1).float()
+        if slot >= 0 and n > 0:
+            state[slot] = S.float()
+    return o_out
+
+
+def delta_step(x, q_off, k_off, v_off, z, a_off, b_off, g_off, decay, dt_bias, q_scale, weight, eps, tok_seq, seq_slot, state, out,
+               H, G, d, dv):
+    for t in range(x.shape[0]):
+        slot = int(seq_slot[int(tok_seq[t])])
+        S = state[slot].double() if slot >= 0 else torch.zeros(H, dv, d, dtype=torch.float64)
+        o = _delta_token(S, x[t], q_off, k_off, v_off, z[t], a_off, b_off, decay, dt_bias, q_scale, H, G, d, dv)
+        if slot >= 0:
+            state[slot] = S.float()
+        gate = z[t, g_off:g_off + H * dv].double().view(H, dv)
+        y = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * weight.double() * gate * torch.sigmoid(gate)
+        out[t] = y.reshape(-1).to(out.dtype)
+    return out

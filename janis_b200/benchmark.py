@@ -110,12 +110,22 @@ def weight_bytes(model, itemsize: int = 2) -> int:
     """Bytes of every tensor a decode step reads once (the tied table counts once: the head reads all of
     it, the embedding a row per sequence)."""
     total = 0
-    for spec in model.tensor_specs().values():
-        n = 1
+    runs = _runs(model)
+    for name, spec in model.tensor_specs().items():
+        n = runs.get(name, 1)
         for s in spec.shape:
             n *= s
         total += n * (4 if len(spec.shape) == 1 else itemsize)
     return total
+
+
+def _runs(model) -> dict:
+    """Tensor name -> how often a step runs the layer it belongs to, for tensors of layers that run more than once."""
+    from .engine.model import _walk
+    times: dict = {}
+    for call in model.schedule:
+        times[call.layer] = times.get(call.layer, 0) + 1
+    return {name: n for layer, n in times.items() if n > 1 for part in _walk(model.blocks[layer]) for name in part.tensor_specs()}
 
 
 def cache_bytes(model, lengths, itemsize: int = 2) -> int:
@@ -140,10 +150,11 @@ def prefill_flops(model, n_tokens: int) -> float:
     """2 M N K of every product of a prompt step of n_tokens that asks for the last logits, plus what each
     layer's mixer says it computes beyond its products (attention: scores and weighted sums)."""
     flops = 0.0
+    runs = _runs(model)
     for name, spec in model.tensor_specs().items():
         if len(spec.shape) == 2 and name not in (getattr(model.embedding, "table_name", None),
                                                     getattr(model.head, "table_name", None)):       # (the head: below)
-            flops += 2.0 * n_tokens * spec.shape[0] * spec.shape[1]
+            flops += 2.0 * n_tokens * spec.shape[0] * spec.shape[1] * runs.get(name, 1)
     for call in model.schedule:
         flops += float(model.blocks[call.layer].mixer.prompt_flops(n_tokens))
     flops += 2.0 * model.hidden * model.vocab          # the head, last position only
@@ -595,6 +606,24 @@ def larulorn_like(gemma: dict, layers: int) -> dict:
             "layers": out}
 
 
+def mugedra_like(gemma: dict, layers: int) -> dict:
+    """A Mugedra configuration with the layer sizes of a Gemma2 one: the same width, heads, head size (for keys and values),
+    feed-forward width and vocabulary; every layer has attention in chunks as long as Gemma2's window (scores capped at 30)
+    beside a gated delta rule whose state is as large as the recurrence of `nosolix_like` (heads of 128 x 128, twice the width in
+    values, two heads a query/key head, a filter of 4 taps); every feed-forward is a mixture of 16 experts of a quarter of the
+    dense width, 4 chosen: as many active feed-forward weights a token as the dense layer."""
+    hd, W, ff = int(gemma["head_dim"]), int(gemma["hidden_size"]), int(gemma["intermediate_size"])
+    left = {"heads": gemma["num_attention_heads"], "kv_heads": gemma["num_key_value_heads"], "dim": hd, "vdim": hd,
+            "scale": hd ** -0.5, "softcap": 30.0, "mask": {"size": int(gemma.get("sliding_window", 4096))},
+            "rot": {"base": 10000.0, "dims": hd, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    kv = max(1, W // 128)
+    right = {"heads": 2 * kv, "kv_heads": kv, "dim": 128, "vdim": 128, "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": max(8, ff // 4 // 8 * 8)}, "router": {"experts": 16, "top": 4}}
+    out = [{"type": "parallel", "mixer": {"left": copy.deepcopy(left), "right": dict(right)}, "mlp": copy.deepcopy(moe)}
+           for _ in range(layers)]
+    return {"architecture": "Mugedra", "vocab": gemma["vocab_size"], "width": W, "norm": {"eps": 1e-6}, "layers": out}
+
+
 _TIMED = {"sigalorn": ("talk_attention", "qkv_rotate_store", "gla_scan", "head_norm_gate", "bias_act", "add_rmsnorm", "rmsnorm"),
           "gemma2": ("attn_prefill", "attn_decode", "rope_store", "gemv_rope_store", "gated_act"),
           "nosolix": ("talk_attention", "talk_attention_rows", "attn_prefill_rows", "attn_decode_rows", "qkv_rotate_store", "selective_scan", "causal_conv_silu", "gate_group_norm",
@@ -605,6 +634,8 @@ _TIMED = {"sigalorn": ("talk_attention", "qkv_rotate_store", "gla_scan", "head_n
           "larulorn": ("talk_attention", "talk_attention_rows", "attn_prefill_rows", "attn_decode_rows", "qkv_rotate_store", "causal_conv_silu", "head_linear",
                        "gated_recurrence_scan", "gated_recurrence_rows", "gate_place", "moe_route", "moe_relu2", "gated_act",
                        "add_rmsnorm", "rmsnorm"),
+          "mugedra": ("talk_attention", "talk_attention_rows", "attn_prefill_rows", "attn_decode_rows", "qkv_rotate_store", "causal_conv_silu",
+                      "delta_scan", "delta_step", "head_norm_gate", "sigmoid_gate", "moe_route", "moe_expert_act", "stream_norm"),
           "vivazen": ("talk_attention", "talk_attention_rows", "qkv_conv_norm_store", "latent_rotate_store", "head_linear", "group_norm", "round_rows",
                       "sigmoid_gate", "gated_act")}
 
@@ -612,6 +643,7 @@ _TIMED = {"sigalorn": ("talk_attention", "qkv_rotate_store", "gla_scan", "head_n
 def _plain_kernel_bytes(model, rows: int) -> dict:
     """Bytes that the kernels between a design's products must move in a step of `rows` tokens in bfloat16, by name: every
     input read once, every output written once (the recurrence: its inputs, its output and its float32 gates)."""
+    from .parts.delta_rule import GatedDeltaRule
     from .parts.feedforward import DenseMLP, GatedMLP
     from .parts.gated_recurrence import GatedRecurrenceMixer
     from .parts.moe import RoutedExperts
@@ -628,6 +660,10 @@ def _plain_kernel_bytes(model, rows: int) -> dict:
             if isinstance(m, GatedRecurrenceMixer):
                 add("causal_conv_silu", 4 * m.width)
                 add("gated_recurrence_scan", (2 + 8 + 2 + 2) * m.width)                 # u, two float logits, the branch, the result
+            elif isinstance(m, GatedDeltaRule):
+                add("causal_conv_silu", 4 * m.channels)
+                add("delta_scan", 2 * m.channels + 4 * m.n_heads + 4 * m.n_heads * m.value_dim)      # q, k, v; two logits a head; the float output
+                add("head_norm_gate", (4 + 2 + 2) * m.n_heads * m.value_dim)
             elif isinstance(m, SelectiveScanMixer):
                 add("causal_conv_silu", 4 * m.inner)
                 add("selective_scan", (2 + 2 + 2 + 2) * m.inner + 4 * m.state)           # u, dt, z, the result; B and C
@@ -635,9 +671,13 @@ def _plain_kernel_bytes(model, rows: int) -> dict:
                 add("causal_conv_silu", 4 * m.conv_channels)
                 add("selective_scan", (2 + 4) * m.inner + 2 * m.n_heads + 4 * m.groups * m.state)
                 add("gate_group_norm", (4 + 2 + 2) * m.inner)
-            if "g" in getattr(m, "names", {}) and hasattr(m, "value_dim") and hasattr(m, "n_heads"):
+            if "g" in getattr(m, "names", {}) and hasattr(m, "n_kv_heads"):
                 add("gate_place" if joined else "sigmoid_gate", 6 * m.n_heads * m.value_dim)
         f = getattr(block, "feed_forward", None)
+        if getattr(block, "mixer_scale", None) is not None:          # the stream read and written, the branches, the next norm's output
+            add("stream_norm", (8 + 2 * len(getattr(block.mixer, "branches", (0,))) + 2) * model.hidden)
+            if f is not None:
+                add("stream_norm", (8 + 2 + 2) * model.hidden)
         if isinstance(f, RoutedExperts):
             add("moe_relu2" if f.act == "relu2" else "moe_expert_act", (4 if f.act == "relu2" else 6) * f.total_ff)
         elif isinstance(f, GatedMLP):
@@ -717,8 +757,8 @@ def _measure_design(raw: dict, kind: str, pk: dict, prefill_tokens: int, batch: 
         att_name = "attn_prefill_rows"
     if kernels["decode_us"].get("attn_decode_rows"):
         dec_name = "attn_decode_rows"
-    scan_name = {"nosolix": "selective_scan", "dekutar": "mlstm_scan", "larulorn": "gated_recurrence_scan"}.get(kind, "gla_scan")
-    scan_decode = "gated_recurrence_rows" if kind == "larulorn" else scan_name
+    scan_name = {"nosolix": "selective_scan", "dekutar": "mlstm_scan", "larulorn": "gated_recurrence_scan", "mugedra": "delta_scan"}.get(kind, "gla_scan")
+    scan_decode = {"larulorn": "gated_recurrence_rows", "mugedra": "delta_step"}.get(kind, scan_name)
     roof = {}
     if kernels["prefill_us"].get(att_name):
         roof["attention_prefill_frac_of_bf16_peak"] = round(att_flops / (kernels["prefill_us"][att_name] * 1e-6) / (pk["bf16_tflops"] * 1e12), 5)
@@ -731,7 +771,7 @@ def _measure_design(raw: dict, kind: str, pk: dict, prefill_tokens: int, batch: 
         roof["recurrence_prefill_tflops_fp32"] = round(gla_flops / (kernels["prefill_us"][scan_name] * 1e-6) / 1e12, 3)
     if kernels["decode_us"].get(scan_decode):
         roof["recurrence_decode_frac_of_copy_bandwidth"] = round(state_bytes / (kernels["decode_us"][scan_decode] * 1e-6) / 1e9 / pk["hbm_gbs"], 5)
-    if kind in ("nosolix", "larulorn"):
+    if kind in ("nosolix", "larulorn", "mugedra"):
         for nm, nbytes in _plain_kernel_bytes(model, prefill_tokens).items():
             if kernels["prefill_us"].get(nm):
                 roof[f"{nm}_prefill_frac_of_copy_bandwidth"] = round(nbytes / (kernels["prefill_us"][nm] * 1e-6) / 1e9 / pk["hbm_gbs"], 5)
@@ -779,7 +819,7 @@ def compare(sizes=("gemma2-2b", "gemma2-9b", "gemma2-27b"), layers: int = 4, pre
     weights: prompt tokens a second, decode tokens a second, and the device time of each design's own kernels in
     one prompt step and one decode step with what fraction of the roofline that is."""
     pk, pk_kind = peaks()
-    beside = {"larulorn": "nosolix", "sigalorn": "gemma2"}.get(design, "sigalorn")
+    beside = {"larulorn": "nosolix", "mugedra": "nosolix", "sigalorn": "gemma2"}.get(design, "sigalorn")
     rec = {"compare": f"{design} beside {beside}", "dtype": "bf16", "data": "synthetic",
            "peaks": pk_kind, "prefill_tokens": prefill_tokens, "batch": batch, "context": context, "steps": steps, "sizes": {}}
     for name in sizes:
@@ -799,6 +839,11 @@ def compare(sizes=("gemma2-2b", "gemma2-9b", "gemma2-27b"), layers: int = 4, pre
             rec["sizes"][name] = {
                 "nosolix": _measure_design(nosolix_like(gemma, layers), "nosolix", pk, prefill_tokens, batch, context, steps, warmup),
                 "larulorn": _measure_design(larulorn_like(gemma, layers), "larulorn", pk, prefill_tokens, batch, context, steps, warmup)}
+            continue
+        if design == "mugedra":      # beside the design it is closest to: attention beside a recurrence, normed and averaged; routed experts
+            rec["sizes"][name] = {
+                "nosolix": _measure_design(nosolix_like(gemma, layers), "nosolix", pk, prefill_tokens, batch, context, steps, warmup),
+                "mugedra": _measure_design(mugedra_like(gemma, layers), "mugedra", pk, prefill_tokens, batch, context, steps, warmup)}
             continue
         if design == "nosolix":      # beside the closest design the library has: recurrent layers between attention over a limited span
             rec["sizes"][name] = {
@@ -832,9 +877,9 @@ def main(argv=None) -> int:
                     "instead of sequences that all reach --context")
     ap.add_argument("--profile", choices=["decode", "prefill"], default="",
                     help="open the CUDA profiler range around two timed decode steps, or the last prompt step")
-    ap.add_argument("--compare", choices=["sigalorn", "nosolix", "vivazen", "dekutar", "larulorn"], default="",
-                    help="instead of the benchmark: Sigalorn beside Gemma2, Nosolix, Vivazen or Dekutar beside Sigalorn, or Larulorn beside "
-                    "Nosolix, at equal layer sizes (prompt and decode throughput, and each design's own kernels against their rooflines); "
+    ap.add_argument("--compare", choices=["sigalorn", "nosolix", "vivazen", "dekutar", "larulorn", "mugedra"], default="",
+                    help="instead of the benchmark: Sigalorn beside Gemma2, Nosolix, Vivazen or Dekutar beside Sigalorn, or Larulorn or Mugedra "
+                    "beside Nosolix, at equal layer sizes (prompt and decode throughput, and each design's own kernels against their rooflines); "
                     "--config picks one size")
     a = ap.parse_args(argv)
     if a.impl == "reference":

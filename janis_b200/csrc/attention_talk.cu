@@ -190,7 +190,11 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
     grid_dependency_wait();
     T* row = rows + (size_t)t * row_elems;
     float* inv_s = reinterpret_cast<float*>(turn_s + hq);            // 1 / root mean square of every head of q and k
-    if (ex.q_norm != nullptr) {
+    // heads that turn whole and whose items (a power of two of them) lie in one warp: the items' threads add the squares up
+    // among themselves; other heads are read once more before
+    const int head_items = hq / V;
+    const bool among = ex.q_norm != nullptr && rot == d && head_items > 0 && head_items <= 32 && (head_items & (head_items - 1)) == 0;
+    if (ex.q_norm != nullptr && !among) {
         for (int head = tid >> 5; head < n_heads; head += nt >> 5) {
             float ss = 0.f;
             for (int c = (tid & 31) * V; c < d; c += 32 * V) {
@@ -204,10 +208,9 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
         }
         __syncthreads();
     }
-    auto norm_head = [&](float (&x)[V], int head, int i) {
+    auto norm_head = [&](float (&x)[V], int head, int i, float inv) {
         if (ex.q_norm == nullptr) return;
         const float* wn = (head < H ? ex.q_norm : ex.k_norm) + i;
-        const float inv = inv_s[head];
 #pragma unroll
         for (int e = 0; e < V; e += 4) {
             float b[4];
@@ -238,8 +241,20 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
             Vec16<T>::load(row + at + hq, b);
             add_bias(a, at);
             add_bias(b, at + hq);
-            norm_head(a, head, i);
-            norm_head(b, head, i + hq);
+            float inv = 1.f;
+            if (among) {
+                const int lane = tid & 31;
+                const unsigned mask = head_items == 32 ? 0xffffffffu : ((1u << head_items) - 1) << (lane & ~(head_items - 1));
+                float ss = 0.f;
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss = fmaf(a[e], a[e], fmaf(b[e], b[e], ss));
+                for (int off = head_items >> 1; off > 0; off >>= 1) ss += __shfl_xor_sync(mask, ss, off);
+                inv = 1.0f / sqrtf(ss / (float)d + ex.norm_eps);
+            } else if (ex.q_norm != nullptr) {
+                inv = inv_s[head];
+            }
+            norm_head(a, head, i, inv);
+            norm_head(b, head, i + hq, inv);
 #pragma unroll
             for (int e = 0; e < V; ++e) {
                 const float2 sc = turn_s[i + e];
@@ -261,7 +276,7 @@ qkv_rotate_store_vec_kernel(T* __restrict__ rows, int row_elems, const int* __re
             Vec16<T>::load(row + at, a);
             if (ex.bias != nullptr || ex.q_norm != nullptr) {
                 add_bias(a, at);
-                norm_head(a, head, c);
+                norm_head(a, head, c, ex.q_norm != nullptr ? inv_s[head] : 1.f);
                 Vec16<T>::store(row + at, a);
             }
             if (head >= H && kdst != nullptr) Vec16<T>::store(kdst + (size_t)(head - H) * JANIS_PAGE * d + c, a);

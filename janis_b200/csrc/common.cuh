@@ -87,8 +87,8 @@ inline int& overlap_launches() {
 
 // Launch with the attribute above, and as thread-block clusters of `cluster` CTAs when cluster > 1.
 template <typename... KArgs, typename... Args>
-inline int launch_kernel(const char* what, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
-                         cudaStream_t stream, int cluster, Args... args) {
+inline int launch_kernel_as(bool early, const char* what, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                            cudaStream_t stream, int cluster, Args... args) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = block;
@@ -103,7 +103,7 @@ inline int launch_kernel(const char* what, void (*kernel)(KArgs...), dim3 grid, 
         attr[n].val.clusterDim.z = 1;
         ++n;
     }
-    if (overlap_launches()) {
+    if (early && overlap_launches()) {
         attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
         attr[n].val.programmaticStreamSerializationAllowed = 1;
         ++n;
@@ -121,6 +121,20 @@ inline int launch_kernel(const char* what, void (*kernel)(KArgs...), dim3 grid, 
 __host__ __device__ __forceinline__ int first_seen(int pos, int window) {
     if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
     return window < 0 ? pos - pos % -window : 0;
+}
+
+template <typename... KArgs, typename... Args>
+inline int launch_kernel(const char* what, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                         cudaStream_t stream, int cluster, Args... args) {
+    return launch_kernel_as(true, what, kernel, grid, block, smem, stream, cluster, args...);
+}
+
+// The same for a kernel of few CTAs that run long: launched once its predecessor is over.  CTAs that arrive while others still
+// hold most SMs pile up on the SMs that are free just then, and stay there.
+template <typename... KArgs, typename... Args>
+inline int launch_kernel_after(const char* what, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                               cudaStream_t stream, int cluster, Args... args) {
+    return launch_kernel_as(false, what, kernel, grid, block, smem, stream, cluster, args...);
 }
 
 // Where a multi-token step finds the keys and values of positions that earlier steps stored: the paged cache line

@@ -73,6 +73,7 @@ delta_coef_kernel(const T* __restrict__ x, const T* __restrict__ z, DeltaShape s
 #pragma unroll
         for (int j = 0; j < DELTA_BLOCK; ++j) kk[i][j] = kq[i][j] = 0.f;
     }
+#pragma unroll 2
     for (int c = lane; c < s.d; c += 32) {
         float kv[DELTA_BLOCK], qv[DELTA_BLOCK];
 #pragma unroll
@@ -109,27 +110,28 @@ delta_coef_kernel(const T* __restrict__ x, const T* __restrict__ z, DeltaShape s
         k_inv[i] = 1.0f / sqrtf(kk[i][i] + DELTA_UNIT_EPS);
         q_inv[i] = s.q_scale / sqrtf(qq[i] + DELTA_UNIT_EPS);
     }
-    const int rep = s.H / s.G;
-    for (int r = lane; r < rep; r += 32) {
-        const int h = kvh * rep + r;
-        float gm1[DELTA_BLOCK], beta[DELTA_BLOCK], till[DELTA_BLOCK], Gm1[DELTA_BLOCK];
-        float run = 0.f;                     // G_i - 1
+    // a lane per (head, token of the block)
+    const int rep = s.H / s.G, me = lane & (DELTA_BLOCK - 1);
+    for (int r0 = 0; r0 < rep; r0 += 32 / DELTA_BLOCK) {
+        const int r = r0 + lane / DELTA_BLOCK, h = kvh * rep + min(r, rep - 1);
+        float own = 0.f, beta = 0.f;
+        if (me < n) delta_gates(z + (size_t)(t + me) * s.z_elems, s, h, decay[h], dt_bias[h], own, beta);
+        float gm1[DELTA_BLOCK];              // g - 1 of every token of the block (0 beyond its end)
+#pragma unroll
+        for (int i = 0; i < DELTA_BLOCK; ++i) gm1[i] = __shfl_sync(0xffffffffu, own, i, DELTA_BLOCK);
+        float till = 1.f, all = 0.f, Gm1 = 0.f;          // c_lj, G_l - 1, G_i - 1
 #pragma unroll
         for (int i = 0; i < DELTA_BLOCK; ++i) {
-            gm1[i] = beta[i] = 0.f;
-            if (i < n) delta_gates(z + (size_t)(t + i) * s.z_elems, s, h, decay[h], dt_bias[h], gm1[i], beta[i]);
-            run = fmaf(run, gm1[i], run) + gm1[i];
-            Gm1[i] = run;
+            all = fmaf(all, gm1[i], all) + gm1[i];
+            if (i == me) Gm1 = all;
+            if (i > me) till = fmaf(till, gm1[i], till);
         }
-        float back = 1.f;                    // c_lj
-#pragma unroll
-        for (int i = DELTA_BLOCK - 1; i >= 0; --i) {
-            till[i] = back;
-            back = fmaf(back, gm1[i], back);
-        }
+        if (me >= n || r >= rep) continue;
+        float4* dst = reinterpret_cast<float4*>(coef + ((size_t)(t + me) * s.H + h) * DELTA_COEF);
+        const float G = 1.0f + Gm1;
 #pragma unroll
         for (int i = 0; i < DELTA_BLOCK; ++i) {
-            if (i >= n) break;
+            if (i != me) continue;
             float A[3] = {0.f, 0.f, 0.f}, B[DELTA_BLOCK] = {0.f, 0.f, 0.f, 0.f};
             float c = 1.f;                   // c_ij
 #pragma unroll
@@ -138,11 +140,9 @@ delta_coef_kernel(const T* __restrict__ x, const T* __restrict__ z, DeltaShape s
                 if (j < i) A[j] = c * kk[i][j] * k_inv[i] * k_inv[j];
                 c = fmaf(c, gm1[j], c);
             }
-            float4* dst = reinterpret_cast<float4*>(coef + ((size_t)(t + i) * s.H + h) * DELTA_COEF);
-            const float G = 1.0f + Gm1[i];
-            dst[0] = make_float4(G * k_inv[i], beta[i], A[0], A[1]);
+            dst[0] = make_float4(G * k_inv[i], beta, A[0], A[1]);
             dst[1] = make_float4(A[2], B[0], B[1], B[2]);
-            dst[2] = make_float4(B[3], till[i] * k_inv[i], G * q_inv[i], Gm1[DELTA_BLOCK - 1]);
+            dst[2] = make_float4(B[3], till * k_inv[i], G * q_inv[i], all);
         }
     }
 }
@@ -150,23 +150,25 @@ delta_coef_kernel(const T* __restrict__ x, const T* __restrict__ z, DeltaShape s
 // grid (sequences, heads, ceil(dv / (8 CPT))); 128 threads: thread = (group of CPT columns, ks), ks fastest.  Lane ks holds
 // key channels ks * DPT .. ks * DPT + DPT - 1 of its columns (channels beyond d hold zeros).  A tile of tokens' q and k lie
 // in shared memory as runs of DPT floats, each followed by 4 floats of padding, so that the lanes' 16-byte reads fall into
-// different banks; the next tile's travel through registers meanwhile.  Tokens beyond the sequence's end are zeros with
+// different banks; the next tile's travel through registers meanwhile, as they are stored (a conversion would wait for
+// them on the spot).  VEC: bfloat16 rows that allow loads of 8 channels.  Tokens beyond the sequence's end are zeros with
 // G = 1, which change nothing.
-template <typename T, int DPT, int CPT>
-__global__ void __launch_bounds__(DELTA_NT)
+template <typename T, int DPT, int CPT, bool VEC>
+__global__ void __launch_bounds__(DELTA_NT, DPT <= 8 ? 4 : 1)
 delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict__ coef, const int* __restrict__ seq_slot,
                   const int* __restrict__ seq_first_row, const int* __restrict__ seq_start, const int* __restrict__ seq_end,
                   float* __restrict__ state, float* __restrict__ o_out) {
     constexpr int RUN = DPT + 4, TOK = DELTA_KS * RUN;
     constexpr int TT = DPT >= 16 ? 8 : 16;                     // tokens staged per round
     constexpr int COLS = DELTA_GROUPS * CPT, WIDTH = DELTA_KS * DPT, NB = DELTA_BLOCK;
-    constexpr int PER = TT * WIDTH / DELTA_NT, CH = WIDTH / 8;
+    constexpr bool KEEP = DPT <= 8;                            // the block's keys stay in registers from the products to the update
+    constexpr int PER = TT * WIDTH / DELTA_NT;
     constexpr int VPER = (TT * COLS + DELTA_NT - 1) / DELTA_NT, C4 = TT * DELTA_COEF / 4;
     static_assert(C4 <= DELTA_NT, "a thread carries one piece of the coefficients");
     __shared__ __align__(16) float q_s[TT * TOK];
     __shared__ __align__(16) float k_s[TT * TOK];
     __shared__ __align__(16) float c_s[TT * DELTA_COEF];
-    __shared__ float v_s[TT * COLS];
+    __shared__ __align__(16) float v_s[TT * COLS];
     const int d = s.d, dv = s.dv, H = s.H;
     const int seq = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * COLS, kvh = h / (H / s.G);
     const int tid = threadIdx.x, ks = tid % DELTA_KS, grp = tid / DELTA_KS, lane = tid & 31;
@@ -185,42 +187,28 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
             S[c][ii] = (st != nullptr && col < dv && i < d) ? st[(size_t)col * d + i] : 0.f;
         }
     }
-    float qv[PER], kv[PER], vv[VPER];
+    constexpr int PIECE = VEC ? 8 : 1, NP = PER / PIECE;
+    typedef typename std::conditional<VEC, uint4, T>::type Raw;
+    Raw qv[NP], kv[NP];
+    T vv[VPER];
+    const T zero = from_float<T>(0.f);
     float4 cf = make_float4(0.f, 0.f, 0.f, 0.f);
-    // 16-byte loads (8 channels of one token a piece) where the rows allow it, else element by element
-    const bool vec = DPT >= 8 && sizeof(T) == 2 && d % 8 == 0 && s.x_elems % 8 == 0 && s.q_off % 8 == 0 && s.k_off % 8 == 0 &&
-                     (((uintptr_t)x) & 15) == 0;
     auto fetch = [&](int t0) {
-        if (vec) {
 #pragma unroll
-            for (int e = 0; e < PER / 8; ++e) {
-                const int u = tid + e * DELTA_NT, tt = u / CH, c0 = (u % CH) * 8;
-#pragma unroll
-                for (int j = 0; j < 8; ++j) qv[e * 8 + j] = kv[e * 8 + j] = 0.f;
-                if (t0 + tt < n_tok && c0 < d) {
-                    const T* row = x + (size_t)(row0 + t0 + tt) * s.x_elems + kvh * d + c0;
-                    Vec16<T>::load(row + s.q_off, &qv[e * 8]);      // (Vec16<bf16>: 8 values; this path is bfloat16 only)
-                    Vec16<T>::load(row + s.k_off, &kv[e * 8]);
-                }
-            }
-        } else {
-#pragma unroll
-            for (int e = 0; e < PER; ++e) {
-                const int u = tid + e * DELTA_NT, tt = u / WIDTH, c = u % WIDTH;
-                qv[e] = kv[e] = 0.f;
-                if (t0 + tt < n_tok && c < d) {
-                    const T* row = x + (size_t)(row0 + t0 + tt) * s.x_elems + kvh * d + c;
-                    qv[e] = to_float(row[s.q_off]);
-                    kv[e] = to_float(row[s.k_off]);
-                }
+        for (int e = 0; e < NP; ++e) {
+            const int u = (tid + e * DELTA_NT) * PIECE, tt = u / WIDTH, c = u % WIDTH;
+            qv[e] = kv[e] = Raw{};
+            if (t0 + tt < n_tok && c < d) {
+                const T* row = x + (size_t)(row0 + t0 + tt) * s.x_elems + kvh * d + c;
+                qv[e] = *reinterpret_cast<const Raw*>(row + s.q_off);
+                kv[e] = *reinterpret_cast<const Raw*>(row + s.k_off);
             }
         }
 #pragma unroll
         for (int e = 0; e < VPER; ++e) {
             const int u = tid + e * DELTA_NT, tt = u / COLS, c = col0 + u % COLS;
-            vv[e] = 0.f;
-            if (u < TT * COLS && t0 + tt < n_tok && c < dv)
-                vv[e] = to_float(x[(size_t)(row0 + t0 + tt) * s.x_elems + s.v_off + h * dv + c]);
+            vv[e] = zero;
+            if (u < TT * COLS && t0 + tt < n_tok && c < dv) vv[e] = x[(size_t)(row0 + t0 + tt) * s.x_elems + s.v_off + h * dv + c];
         }
         if (tid < C4) {
             constexpr int P = DELTA_COEF / 4;
@@ -230,9 +218,21 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
                 cf = reinterpret_cast<const float4*>(coef + ((size_t)(row0 + t0 + tt) * H + h) * DELTA_COEF)[tid % P];
         }
     };
+    // one piece of a token's channels, from channel c on, into the token's runs
+    auto put_piece = [](float* tok, int c, const Raw& raw) {
+        if constexpr (VEC) {
+            float f[8];
+            Vec16<bf16>::load(reinterpret_cast<const bf16*>(&raw), f);
+#pragma unroll
+            for (int e = 0; e < 8; e += 4)
+                *reinterpret_cast<float4*>(tok + ((c + e) / DPT) * RUN + (c + e) % DPT) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+        } else {
+            tok[(c / DPT) * RUN + c % DPT] = to_float(raw);
+        }
+    };
     // which of a block's sums this lane ends up with: column, products with q (or with k), token
     const int my_c = CPT == 2 ? ks >> 3 : 0;
-    const bool my_q = CPT == 2 ? ((ks >> 2) & 1) != 0 : (ks >> 3) != 0;
+    const bool my_q = (CPT == 2 ? (ks >> 2) & 1 : ks >> 3) != 0;
     const int my_i = CPT == 2 ? ks & 3 : (ks >> 1) & 3;
     const int my_col = col0 + grp * CPT + my_c;
     const bool writer = my_q && my_col < dv && (CPT == 2 || (ks & 1) == 0);
@@ -240,24 +240,14 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
     for (int t0 = 0; t0 < n_tok; t0 += TT) {
         __syncthreads();                       // the tile before has been read
 #pragma unroll
-        for (int e = 0; e < PER; ++e) {
-            int tt, c;
-            if (vec) {
-                const int u = tid + (e / 8) * DELTA_NT;
-                tt = u / CH;
-                c = (u % CH) * 8 + e % 8;
-            } else {
-                const int u = tid + e * DELTA_NT;
-                tt = u / WIDTH;
-                c = u % WIDTH;
-            }
-            const int at = tt * TOK + (c / DPT) * RUN + c % DPT;
-            q_s[at] = qv[e];
-            k_s[at] = kv[e];
+        for (int e = 0; e < NP; ++e) {
+            const int u = (tid + e * DELTA_NT) * PIECE, tt = u / WIDTH, c = u % WIDTH;
+            put_piece(q_s + tt * TOK, c, qv[e]);
+            put_piece(k_s + tt * TOK, c, kv[e]);
         }
 #pragma unroll
         for (int e = 0; e < VPER; ++e)
-            if (tid + e * DELTA_NT < TT * COLS) v_s[tid + e * DELTA_NT] = vv[e];
+            if (tid + e * DELTA_NT < TT * COLS) v_s[tid + e * DELTA_NT] = to_float(vv[e]);
         if (tid < C4) reinterpret_cast<float4*>(c_s)[tid] = cf;
         __syncthreads();
         if (t0 + TT < n_tok) fetch(t0 + TT);
@@ -266,6 +256,7 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
             if (t0 + b >= n_tok) break;
             // the block's products with the state before it
             float sum[8 * CPT];                // [column][k, q][token]
+            float kr[KEEP ? NB : 1][DPT];      // this lane's run of the block's keys, for the update below
 #pragma unroll
             for (int v = 0; v < 8 * CPT; ++v) sum[v] = 0.f;
 #pragma unroll
@@ -274,6 +265,10 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
                 for (int i = 0; i < NB; ++i) {
                     const float4 k4 = reinterpret_cast<const float4*>(k_s + (b + i) * TOK + ks * RUN)[i4];
                     const float4 q4 = reinterpret_cast<const float4*>(q_s + (b + i) * TOK + ks * RUN)[i4];
+                    if (KEEP) {
+                        float* k_ = &kr[KEEP ? i : 0][4 * i4];
+                        k_[0] = k4.x; k_[1] = k4.y; k_[2] = k4.z; k_[3] = k4.w;
+                    }
 #pragma unroll
                     for (int c = 0; c < CPT; ++c) {
                         const float* Sc = &S[c][4 * i4];
@@ -307,20 +302,19 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
             }
             const float mine = sum[0];
             // every lane solves for the block's u
+            const float4* cb = reinterpret_cast<const float4*>(c_s + b * DELTA_COEF);
             float u[CPT][NB];
 #pragma unroll
-            for (int c = 0; c < CPT; ++c) {
-                float p[NB];
+            for (int i = 0; i < NB; ++i) {
+                const float4 c0 = cb[3 * i];
+                const float A[3] = {c0.z, c0.w, i == 3 ? c_s[(b + i) * DELTA_COEF + 4] : 0.f};
 #pragma unroll
-                for (int i = 0; i < NB; ++i)
-                    p[i] = __shfl_sync(0xffffffffu, mine, (lane & 16) | (CPT == 2 ? c * 8 + i : 2 * i));
+                for (int c = 0; c < CPT; ++c) {
+                    const float p = __shfl_sync(0xffffffffu, mine, (lane & 16) | (CPT == 2 ? c * 8 + i : 2 * i));
+                    float r = fmaf(-c0.x, p, v_s[(b + i) * COLS + grp * CPT + c]);
 #pragma unroll
-                for (int i = 0; i < NB; ++i) {
-                    const float* ci = c_s + (b + i) * DELTA_COEF;
-                    float r = fmaf(-ci[0], p[i], v_s[(b + i) * COLS + grp * CPT + c]);
-#pragma unroll
-                    for (int j = 0; j < i; ++j) r = fmaf(-ci[2 + j], u[c][j], r);
-                    u[c][i] = ci[1] * r;
+                    for (int j = 0; j < i; ++j) r = fmaf(-A[j], u[c][j], r);
+                    u[c][i] = c0.y * r;
                 }
             }
             if (writer && t0 + b + my_i < n_tok) {
@@ -330,11 +324,14 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
                 for (int j = 0; j < NB; ++j) o = fmaf(ci[5 + j], CPT == 2 && my_c ? u[CPT - 1][j] : u[0][j], o);
                 o_out[(size_t)(row0 + t0 + b + my_i) * H * dv + h * dv + my_col] = o;
             }
-            const float gm1 = c_s[b * DELTA_COEF + 11];
+            float gm1 = 0.f;
 #pragma unroll
-            for (int c = 0; c < CPT; ++c)
+            for (int j = 0; j < NB; ++j) {
+                const float4 c2 = cb[3 * j + 2];
+                if (j == 0) gm1 = c2.w;
 #pragma unroll
-                for (int j = 0; j < NB; ++j) u[c][j] *= c_s[(b + j) * DELTA_COEF + 9];
+                for (int c = 0; c < CPT; ++c) u[c][j] *= c2.y;
+            }
 #pragma unroll
             for (int i4 = 0; i4 < DPT / 4; ++i4) {
                 float add[CPT][4];
@@ -344,14 +341,18 @@ delta_scan_kernel(const T* __restrict__ x, DeltaShape s, const float* __restrict
                     for (int e = 0; e < 4; ++e) add[c][e] = S[c][4 * i4 + e] * gm1;
 #pragma unroll
                 for (int j = 0; j < NB; ++j) {
-                    const float4 k4 = reinterpret_cast<const float4*>(k_s + (b + j) * TOK + ks * RUN)[i4];
+                    float k_[4];
+                    if (KEEP) {
 #pragma unroll
-                    for (int c = 0; c < CPT; ++c) {
-                        add[c][0] = fmaf(k4.x, u[c][j], add[c][0]);
-                        add[c][1] = fmaf(k4.y, u[c][j], add[c][1]);
-                        add[c][2] = fmaf(k4.z, u[c][j], add[c][2]);
-                        add[c][3] = fmaf(k4.w, u[c][j], add[c][3]);
+                        for (int e = 0; e < 4; ++e) k_[e] = kr[KEEP ? j : 0][4 * i4 + e];
+                    } else {
+                        const float4 k4 = reinterpret_cast<const float4*>(k_s + (b + j) * TOK + ks * RUN)[i4];
+                        k_[0] = k4.x; k_[1] = k4.y; k_[2] = k4.z; k_[3] = k4.w;
                     }
+#pragma unroll
+                    for (int c = 0; c < CPT; ++c)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) add[c][e] = fmaf(k_[e], u[c][j], add[c][e]);
                 }
 #pragma unroll
                 for (int c = 0; c < CPT; ++c)
@@ -523,23 +524,26 @@ static int delta_prompt_launch(const void* x, const void* z, const DeltaShape& s
     if (launch_kernel("delta_coef", delta_coef_kernel<T>, dim3(n_tok, (s.G + warps - 1) / warps), dim3(warps * 32), 0, stream, 1, (const T*)x,
                       (const T*)z, s, decay, dt_bias, tok_pos, tok_seq, seq_start, seq_end, coef, n_tok))
         return 1;
-    // two columns a group of lanes halve the reads from shared memory and the exchanges a column; with few heads one column
-    // a group keeps more SMs busy
-    const bool two = form ? form == 2 : (long long)n_seq * s.H * ((s.dv + 15) / 16) >= 120;
+    // two columns a group of lanes halve the reads from shared memory and the exchanges a column; where one column a group
+    // leaves every CTA an SM of its own that is faster still
+    const bool two = form ? form == 2 : (long long)n_seq * s.H * ((s.dv + DELTA_GROUPS - 1) / DELTA_GROUPS) > 148;
     const int cols = DELTA_GROUPS * (two ? 2 : 1);
     const dim3 grid(n_seq, s.H, (s.dv + cols - 1) / cols), block(DELTA_NT);
+    // 16-byte loads (8 channels of one token a piece) where the rows allow it, else element by element
+    const bool vec = sizeof(T) == 2 && s.d % 8 == 0 && s.x_elems % 8 == 0 && s.q_off % 8 == 0 && s.k_off % 8 == 0 && ((uintptr_t)x & 15) == 0;
+#define JANIS_DELTA_LAUNCH(DPT, CPT)                                                                                   \
+    return launch_kernel_after("delta_scan", vec ? delta_scan_kernel<T, DPT, CPT, sizeof(T) == 2> : delta_scan_kernel<T, DPT, CPT, false>, grid, block, 0, stream, 1, (const T*)x, s, (const float*)coef, \
+                         seq_slot, seq_first_row, seq_start, seq_end, state, o_out);
 #define JANIS_DELTA_CASE(DPT)                                                                                          \
     if (s.d <= DELTA_KS * DPT) {                                                                                       \
-        if (two)                                                                                                       \
-            return launch_kernel("delta_scan", delta_scan_kernel<T, DPT, 2>, grid, block, 0, stream, 1, (const T*)x, s, \
-                                 (const float*)coef, seq_slot, seq_first_row, seq_start, seq_end, state, o_out);       \
-        return launch_kernel("delta_scan", delta_scan_kernel<T, DPT, 1>, grid, block, 0, stream, 1, (const T*)x, s,    \
-                             (const float*)coef, seq_slot, seq_first_row, seq_start, seq_end, state, o_out);           \
+        if (two) { JANIS_DELTA_LAUNCH(DPT, 2) }                                                                   \
+        JANIS_DELTA_LAUNCH(DPT, 1)                                                                                     \
     }
     JANIS_DELTA_CASE(4)
     JANIS_DELTA_CASE(8)
     JANIS_DELTA_CASE(16)
 #undef JANIS_DELTA_CASE
+#undef JANIS_DELTA_LAUNCH
     return fail("delta_scan: key size %d is above %d", s.d, DELTA_KS * 16);
 }
 
@@ -554,6 +558,7 @@ JANIS_EXPORT int janis_delta_scan(const void* x, int x_elems, int q_off, int k_o
     if (n_seq <= 0 || n_tok <= 0) return 0;
     const DeltaShape s = {H, G, d, dv, x_elems, q_off, k_off, v_off, z_elems, a_off, b_off, q_scale};
     if (delta_check("delta_scan", s)) return 1;
+    if (form < 0 || form > 2) return fail("delta_scan: %d columns a group of lanes", form);
     if (((uintptr_t)coef) & 15) return fail("delta_scan: the coefficients start on a 16-byte border");
     if (dtype == JANIS_F32)
         return delta_prompt_launch<float>(x, z, s, decay, dt_bias, coef, tok_pos, tok_seq, seq_slot, seq_first_row, seq_start, seq_end,
